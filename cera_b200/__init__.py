@@ -12,3 +12,5 @@ from .ops import (MoeFfn, QuantWeight, Q8Activations, decode_attention, decode_a
                   block_sums, quantize_columns, quantize_q8_0, quantize_weights, rmsnorm, rmsnorm_q8_0, rope, silu_mul,
                   synth_normal)
 from .model import CudaModel, ModelConfig, Role  # noqa: F401
+from .layered import LayeredModel  # noqa: F401
+from .registry import load_model  # noqa: F401

@@ -30,6 +30,18 @@ class Config(C.Structure):
                 ("logit_scale", _f)]
 
 
+class LayerDesc(C.Structure):
+    _fields_ = [("mixer", _i32), ("ff", _i32), ("n_heads", _u32), ("head_dim", _u32), ("rot_dim", _u32), ("value_dim", _u32),
+                ("kv_rank", _u32), ("rope_base", _f), ("attn_scale", _f), ("recurrent_width", _u32), ("ff_width", _u32),
+                ("n_experts", _u32), ("n_used", _u32), ("act_limit", _f), ("act_alpha", _f), ("act_shift", _f),
+                ("router_softmax", _i32), ("router_renorm", _i32), ("weight_input", _i32)]
+
+
+class LayeredConfig(C.Structure):
+    _fields_ = [("n_layers", _u32), ("hidden_size", _u32), ("vocab_size", _u32), ("max_seq_len", _u32), ("norm_eps", _f),
+                ("dtype", _i32), ("device", _i32), ("bigram_buckets", _u32), ("bigram_mul_prev", _u64), ("bigram_mul_cur", _u64)]
+
+
 # name -> (restype, argtypes); every symbol include/cera_cuda.h declares.
 SIGNATURES = {
     "cera_cuda_last_error": (C.c_char_p, []),
@@ -74,6 +86,9 @@ SIGNATURES = {
     "cera_cuda_launch_count": (_u64, [_p]),
     "cera_cuda_model_free": (None, [_p]),
     "cera_cuda_forward_prefill_logits_all": (_i32, [_p, _p, _sz, _sz, _p]),
+    "cera_cuda_forward_prefill_logits_at": (_i32, [_p, _p, _sz, _sz, _p, _sz, _p]),
+    "cera_cuda_model_create_layered": (_i32, [C.POINTER(LayeredConfig), C.POINTER(LayerDesc), C.POINTER(_p)]),
+    "cera_cuda_model_add_expert_tensor": (_i32, [_p, _i32, _i32, _i32, _i32, _sz, _sz, _p, _sz]),
     "cera_cuda_model_attach_lora": (_i32, [_p, _i32, _i32, _sz, _sz, _sz, _p, _p, _f]),
     "cera_cuda_model_detach_lora": (_i32, [_p]),
     "cera_cuda_kv_shift": (_i32, [_p, _sz, _sz]),
@@ -94,7 +109,37 @@ SIGNATURES = {
     "cera_cuda_moe_free": (None, [_p]),
 }
 
+# A library may be built from some of its parts (build.py); one of the others is then absent as a whole, and its calls raise.
+CORE = {"cera_cuda_last_error", "cera_cuda_kernel_status", "cera_cuda_device_count", "cera_cuda_model_add_tensor",
+        "cera_cuda_model_finalize", "cera_cuda_forward", "cera_cuda_forward_greedy", "cera_cuda_generate_greedy",
+        "cera_cuda_forward_prefill", "cera_cuda_forward_prefill_logits_all", "cera_cuda_forward_prefill_logits_at",
+        "cera_cuda_truncate_kv", "cera_cuda_seq_len", "cera_cuda_memory_bytes", "cera_cuda_last_hidden", "cera_cuda_launch_count",
+        "cera_cuda_model_free", "cera_cuda_kv_snapshot_bytes", "cera_cuda_kv_snapshot", "cera_cuda_kv_restore"}
+LAYERED = {"cera_cuda_model_create_layered", "cera_cuda_model_add_expert_tensor"}
+_MARK = {"layered": "cera_cuda_model_create_layered", "quantized": "cera_cuda_model_create"}
+
+
+def part_of(name):
+    return "core" if name in CORE else "layered" if name in LAYERED else "quantized"
+
+
+_PRESENT = {"core"} | {part for part, name in _MARK.items() if hasattr(lib, name)}
+
+
+def has_part(part):
+    return part in _PRESENT
+
+
+def _absent(name, part):
+    def call(*_):
+        raise CeraCudaError(2, f"{name}: this library was built without its {part!r} part (python cera_b200/build.py builds all)")
+    return call
+
+
 for _name, (_res, _args) in SIGNATURES.items():
+    if not has_part(part_of(_name)):
+        setattr(lib, _name, _absent(_name, part_of(_name)))
+        continue
     try:
         _fn = getattr(lib, _name)
     except AttributeError as e:  # the library does not export a declared symbol: stale build

@@ -15,7 +15,12 @@ CSRC = os.path.join(HERE, "csrc")
 OBJ_DIR = os.path.join(HERE, "_obj")
 LIB = os.path.join(HERE, "libcera_cuda.so")
 
-SOURCES = ["runtime.cu", "weight.cu", "quantize.cu", "gemv.cu", "attention.cu", "glue.cu", "convert.cu", "model.cu"]
+# The library's parts: a build may take only what a model needs (bin/trace_run in a fresh checkout); the default is all.
+# Everything that is not listed belongs to "quantized".
+PARTS = {"core": ["runtime.cu", "model.cu", "argmax.cu"],
+         "layered": ["layered.cu", "dense.cu", "dense_gemv.cu", "dense_gemm.cu", "dense_gemm_tc.cu", "mingru.cu", "latent_attention.cu",
+                     "latent_prefill.cu", "moe_route.cu"]}
+ALL_PARTS = ("core", "layered", "quantized")
 # Translation units whose float arithmetic must not be contracted into FMAs.
 NO_FMAD = {"convert.cu"}
 
@@ -44,17 +49,19 @@ def _stale(target, deps):
     return any(os.path.getmtime(d) > t for d in deps)
 
 
-def _sources():
-    extra = [f for f in sorted(os.listdir(CSRC)) if f.endswith(".cu") and f not in SOURCES]
-    return SOURCES + extra
+def _sources(parts):
+    listed = [f for p in PARTS.values() for f in p]
+    rest = [f for f in sorted(os.listdir(CSRC)) if f.endswith(".cu") and f not in listed]
+    # moe_route.cu is shared: part of either build
+    return [f for p in parts for f in (rest + ["moe_route.cu"] if p == "quantized" else PARTS[p])]
 
 
-def build(force=False, verbose=False):
+def build(force=False, verbose=False, parts=ALL_PARTS):
     os.makedirs(OBJ_DIR, exist_ok=True)
     hdrs = _headers()
     jobs = []
     objs = []
-    for src in _sources():
+    for src in dict.fromkeys(_sources(parts)):
         s = os.path.join(CSRC, src)
         o = os.path.join(OBJ_DIR, src.replace(".cu", ".o"))
         objs.append(o)
@@ -76,12 +83,16 @@ def build(force=False, verbose=False):
                     sys.stderr.write(" ".join(cmd[-3:]) + "\n" + r.stdout + r.stderr)
                 if r.returncode:
                     raise RuntimeError("nvcc failed for " + cmd[-3])
-    if jobs or force or _stale(LIB, objs):
+    made_of = os.path.join(OBJ_DIR, "linked.txt")  # the objects the library was linked from
+    before = open(made_of).read().split() if os.path.exists(made_of) else []
+    if jobs or force or _stale(LIB, objs) or before != [os.path.basename(o) for o in objs]:
         cmd = [nvcc()] + ARCH + ["-shared", "-o", LIB] + objs
         r = subprocess.run(cmd, capture_output=True, text=True)
         if r.returncode:
             sys.stderr.write(r.stdout + r.stderr)
             raise RuntimeError("link failed")
+        with open(made_of, "w") as f:
+            f.write("\n".join(os.path.basename(o) for o in objs))
     return LIB
 
 

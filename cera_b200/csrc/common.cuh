@@ -14,6 +14,9 @@ namespace cera {
 // ---- status ---------------------------------------------------------------
 int32_t fail(int32_t code, const char *fmt, ...);
 int32_t check_cuda(cudaError_t e, const char *what);
+// Kernels with bounded waits keep a status word in device memory; the file that owns one registers its reader here
+// (at load time) and cera_cuda_kernel_status ORs them all.
+bool register_kernel_status(uint32_t (*reader)());
 void count_launch(int n = 1);      // bumps the library-wide kernel launch counter
 uint64_t launches_so_far();
 

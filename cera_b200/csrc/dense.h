@@ -1,0 +1,152 @@
+// Dense (bf16 or f32) weights and the operators of models described layer by layer (layered.cu).
+//
+// Conventions: activations are token-major rows; T, the element type of weights and activations, is bf16 or f32
+// (`f32` flags); every row length `ld` is a multiple of 64 elements and the padding is zero, so kernels walk whole
+// 16-byte vectors and padded weight rows produce zeros.  Residual stream, norms, routing, scores, recurrent state: f32.
+#pragma once
+
+#include <cuda_bf16.h>
+
+#include "ops.h"
+
+namespace cera {
+
+struct DenseView {
+    const void *w = nullptr;
+    uint32_t rows = 0, ld = 0;  // [rows][ld], zero-padded
+    int f32 = 0;
+};
+
+inline uint32_t pad_to(uint32_t v, uint32_t a) { return (v + a - 1) / a * a; }
+
+// A norm: g holds one number (per_channel 0) or one per channel (1).
+struct NormView {
+    const float *g = nullptr;
+    int per_channel = 0;
+};
+
+// Index i of a padded axis: groups of `group` source entries become groups of `group_p`, of which the first `seg`
+// entries stay in front and the rest start at seg_p.
+struct PadMap {
+    uint32_t group = 0xFFFFFFFFu, group_p = 0, seg = 0xFFFFFFFFu, seg_p = 0, base = 0;
+    __host__ __device__ uint32_t operator()(uint32_t i) const {
+        const uint32_t g = i / group, r = i - g * group;
+        return base + g * group_p + (r < seg ? r : seg_p + (r - seg));
+    }
+};
+
+// ---- weights (dense.cu) ---------------------------------------------------------------------------------------
+// src [rows][cols] of CERA_TYPE_BF16 / F16 / F32 -> dst element (rmap(row), cmap(col)) of row length ld.
+int32_t launch_place(const void *src, int32_t src_type, size_t rows, size_t cols, void *dst, int dst_f32, size_t ld, const PadMap &rmap,
+                     const PadMap &cmap, cudaStream_t st);
+
+// ---- embedding and norms (dense.cu) ------------------------------------------------------------------------------
+struct BigramParams {
+    uint32_t buckets = 0;  // 0: none
+    uint64_t mul_prev = 0, mul_cur = 0;
+};
+// x[j] = table[token j] (+ bigram row).  tokens[0] is the token before the first one (NO_TOKEN: none), tokens[1 + j] token
+// j; with dyn the step's token and its predecessor are read from the dyn words instead (n == 1).
+int32_t launch_embed_dense(const DenseView &table, const DenseView &bigram, const BigramParams &bp, const uint32_t *tokens, const uint32_t *dyn,
+                           size_t n, float *x, cudaStream_t st);
+// One sublayer boundary for n rows of `width` numbers (row length ld):
+//   y (optional): x += norm_post(sum over picks of y[entry]) with entry = entry_of[j * picks + s], or row j without it
+//   then h = norm_pre(x), as T in h and / or f32 in h32.
+// x_rows (optional): row j of x is x[x_rows[j]] (no residual update then).
+struct ResidualNorm {
+    float *x = nullptr;
+    const float *y = nullptr;
+    const uint32_t *entry_of = nullptr;
+    const float *pick_weight = nullptr;  // multiplies an entry's row
+    uint32_t picks = 1;
+    NormView post, pre;
+    void *h = nullptr;
+    int h_f32 = 0;
+    float *h32 = nullptr;
+    const uint32_t *x_rows = nullptr;
+};
+int32_t launch_residual_norm(const ResidualNorm &p, uint32_t width, uint32_t ld, size_t n, float eps, cudaStream_t st);
+
+// ---- one-column products (dense_gemv.cu) --------------------------------------------------------------------------
+int32_t launch_dense_gemv(const DenseView &w, const void *x, float *y, cudaStream_t st);
+// minGRU decode step: rows [0, wp) z, [wp, 2 wp) candidate, [2 wp, 3 wp) gate of w; updates state, out = state * silu(gate).
+int32_t launch_mingru_step(const DenseView &w, const void *x, const float *z_bias, const float *x_bias, float *state, void *out, cudaStream_t st);
+struct ExpertAct {
+    float limit = 0.0f, alpha = 0.0f, shift = 0.0f;
+};
+struct RouterRule {
+    uint32_t n_expert = 0, n_used = 0;
+    int softmax = 0, renorm = 0, weight_input = 0;
+};
+// Routed feed-forward of one token: picks from the router logits, gate / up rows of the chosen experts through the gated
+// unit into act [n_used][ff_p]; the second call y = sum over picks of down rows.  w_gate_up stacks per expert ff_p gate
+// rows then ff_p up rows, w_down `rows_per_expert` rows per expert.
+int32_t launch_expert_gate_up_step(const DenseView &w_gate_up, const void *x, const float *router_logits, const RouterRule &r, uint32_t ff_p,
+                                   const ExpertAct &a, uint32_t *ids, float *weights, void *act, cudaStream_t st);
+int32_t launch_expert_down_step(const DenseView &w_down, uint32_t rows_per_expert, const void *act, const RouterRule &r, const uint32_t *ids,
+                                const float *weights, float *y, cudaStream_t st);
+
+// ---- many-column products (dense_gemm.cu, dense_gemm_tc.cu) ----------------------------------------------------------
+enum DenseOut { DENSE_F32 = 0, DENSE_T = 1, DENSE_T_TRANSPOSED = 2, DENSE_GATED_UNIT = 3 };
+struct DenseGemm {
+    DenseView w;
+    const void *x = nullptr;  // [n][w.ld]
+    uint32_t n = 0;           // rows of x (grouped: rows of the gathered buffer)
+    int out_kind = DENSE_F32;
+    void *out = nullptr;  // out[j * ldo + row]; transposed: out[row * ldo + j]
+    size_t ldo = 0;
+    // grouped by expert: item (expert, first, count) takes rows [expert * rows_per_expert, + rows_per_expert) of w against
+    // columns [first, first + count)
+    const MoeTile *tiles = nullptr;
+    const uint32_t *n_tiles = nullptr;
+    uint32_t max_tiles = 0, rows_per_expert = 0;
+    // DENSE_GATED_UNIT (grouped): rows_per_expert = 2 ff_p, out [columns][ff_p] of T = unit(scale * gate, scale * up)
+    ExpertAct act;
+    const float *col_scale = nullptr;
+};
+constexpr uint32_t DENSE_GROUP_COLUMNS = 128;  // columns of a grouped item
+int32_t launch_dense_gemm(const DenseGemm &g, cudaStream_t st);
+// The bf16 product on tcgen05 / TMEM.  *taken = false: not its case, nothing launched.
+int32_t launch_dense_gemm_tc(const DenseGemm &g, cudaStream_t st, bool *taken);
+// Columns of a batch in bucket order: g[pos] = h[token], entry_of[pair] = pos, col_scale[pos] = the pair's weight.
+int32_t launch_moe_gather(const void *h, int f32, uint32_t ld, const uint32_t *ids, const float *weights, uint32_t n_used, size_t n, uint32_t *cursor,
+                          uint32_t *entry_of, void *g, float *col_scale, cudaStream_t st);
+
+// ---- minGRU over a prompt portion (mingru.cu) -----------------------------------------------------------------------
+// pre: [n][3 wp] raw z / candidate / gate products; state: [wp], advanced by n positions.
+int32_t launch_mingru_scan(const float *pre, size_t n, uint32_t wp, const float *z_bias, const float *x_bias, float *state, void *out, int f32,
+                           cudaStream_t st);
+
+// ---- latent attention (latent_attention.cu, latent_prefill.cu) --------------------------------------------------------
+struct LatentShape {
+    uint32_t heads = 0, dim = 0, rot = 0, vdim = 0, rank = 0;          // as the model states them
+    uint32_t dim_p = 0, rot_p = 0, vdim_p = 0, rank_p = 0, in_p = 0;    // padded; in_p: row length of the input products
+    __host__ __device__ uint32_t q_ld() const { return heads * (dim_p + rot_p); }
+    __host__ __device__ uint32_t off_c() const { return heads * (dim_p + rot_p); }
+    __host__ __device__ uint32_t off_r() const { return off_c() + rank_p; }
+    __host__ __device__ uint32_t off_g() const { return off_r() + rot_p; }
+    float scale = 0.0f;
+};
+// Input products [n][in_p] = q | latent | rotated key | gate logits.  Normalises the latent, rotates the key part and q,
+// appends both to the cache at positions pos.. (pos_dev: read from device memory, n == 1), q as f32 (q32) and / or T (qt),
+// gate = sigmoid(logit) [n][heads].
+int32_t launch_latent_prepare(const float *in, const LatentShape &s, size_t n, size_t start_pos, const uint32_t *pos_dev, const float *c_norm, float eps,
+                              const float *rope_table, void *cache_c, void *cache_r, int f32, float *q32, void *qt, float *gate, cudaStream_t st);
+// Attention in the latent space for n queries at positions start_pos + j (or *len_dev - 1): q_lat = W_uk^T q, scores
+// against the cached latents, per-split partial sums, merge with the sink, W_uv, gate.  out [n][ldo] of T, heads * vdim_p used.
+struct LatentScratch {
+    float *q_lat = nullptr;  // [queries][heads][rank_p + rot_p]
+    float *part = nullptr;   // [queries][heads][splits][rank_p + 2]
+};
+constexpr uint32_t LATENT_MAX_SPLITS = 64;  // queries * splits of one call never exceed this
+uint32_t latent_splits(size_t n_positions);
+int32_t launch_latent_attention(const float *q32, const LatentShape &s, const DenseView &uk, const DenseView &uv, const void *cache_c, const void *cache_r,
+                                const float *sink, const float *gate, size_t n, size_t start_pos, const uint32_t *len_dev, uint32_t splits,
+                                const LatentScratch &ws, void *out, size_t ldo, cudaStream_t st);
+// Tensor-core attention of a prompt portion: keys and values of the positions [0, start_pos + n) are expanded into k_exp
+// [positions][heads * dim_p] and v_exp [heads * vdim_p][ld_v] (bf16) first.  *taken = false: not its case.
+bool latent_prefill_supports(const LatentShape &s);
+int32_t launch_latent_prefill(const void *qt, const LatentShape &s, const void *k_exp, const void *cache_r, size_t cache_rows, const void *v_exp, size_t ld_v,
+                              const float *sink, const float *gate, size_t n, size_t start_pos, void *out, size_t ldo, cudaStream_t st, bool *taken);
+
+}  // namespace cera

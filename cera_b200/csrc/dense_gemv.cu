@@ -1,0 +1,265 @@
+// One-column products with dense weights: the decode step's projections, with the work that follows them fused where
+// one warp holds all a result needs (the minGRU update, the experts' gated unit, the sum over picks).
+//
+// A row group (R rows that share the activation vector) is walked by WPR warps of a CTA, 16 bytes per lane and row at a
+// time; the first loads are issued before the kernel waits for its predecessor (weights never change).
+#include "dense.cuh"
+#include "moe_route.cuh"
+
+namespace cera {
+
+namespace {
+
+constexpr int GV_WARPS = 8;
+
+template <class T, int R, int U>
+struct RowDot {
+    const T *w[R];
+    uint32_t nv, step, c;
+    uint4 buf[R][U];
+    // part of `parts` warps that share the row; ld elements per row
+    __device__ __forceinline__ void start(uint32_t ld, int part, int parts) {
+        nv = ld / Elem<T>::N;
+        step = 32u * parts;
+        c = part * 32u + (threadIdx.x & 31);
+    }
+    __device__ __forceinline__ void fetch() {
+#pragma unroll
+        for (int u = 0; u < U; ++u)
+            if (c + u * step < nv) {
+#pragma unroll
+                for (int r = 0; r < R; ++r) buf[r][u] = ld_stream(reinterpret_cast<const uint4 *>(w[r]) + c + u * step);
+            }
+    }
+    __device__ __forceinline__ void run(const T *x, float (&acc)[R]) {
+        while (c < nv) {
+#pragma unroll
+            for (int u = 0; u < U; ++u)
+                if (c + u * step < nv) {
+                    float xf[Elem<T>::N], wf[Elem<T>::N];
+                    Elem<T>::unpack(*(reinterpret_cast<const uint4 *>(x) + c + u * step), xf);
+#pragma unroll
+                    for (int r = 0; r < R; ++r) {
+                        Elem<T>::unpack(buf[r][u], wf);
+#pragma unroll
+                        for (int i = 0; i < Elem<T>::N; ++i) acc[r] = fmaf(wf[i], xf[i], acc[r]);
+                    }
+                }
+            c += U * step;
+            fetch();
+        }
+    }
+};
+
+// Sums of R values over the WPR warps of a group; valid in lane 0 of the group's first warp.
+template <int R, int WPR>
+__device__ __forceinline__ void group_sum(float (&acc)[R], float (*red)[R]) {
+#pragma unroll
+    for (int r = 0; r < R; ++r) acc[r] = warp_sum(acc[r]);
+    if (WPR == 1) return;
+    const int warp = threadIdx.x >> 5;
+    if ((threadIdx.x & 31) == 0) {
+#pragma unroll
+        for (int r = 0; r < R; ++r) red[warp][r] = acc[r];
+    }
+    __syncthreads();
+    if (warp % WPR == 0) {
+#pragma unroll
+        for (int r = 0; r < R; ++r) {
+            acc[r] = 0.0f;
+#pragma unroll
+            for (int i = 0; i < WPR; ++i) acc[r] += red[warp + i][r];
+        }
+    }
+}
+
+template <class T, int R, int WPR>
+__global__ void __launch_bounds__(GV_WARPS * 32) gemv_kernel(const T *__restrict__ w, uint32_t rows, uint32_t ld, const T *x, float *y) {
+    __shared__ float red[GV_WARPS][R];
+    pdl_trigger();
+    const int warp = threadIdx.x >> 5;
+    const uint32_t g = blockIdx.x * (GV_WARPS / WPR) + warp / WPR;
+    RowDot<T, R, R == 1 ? 8 : 4> d;
+#pragma unroll
+    for (int r = 0; r < R; ++r) d.w[r] = w + (size_t)min(g * R + r, rows - 1) * ld;
+    d.start(ld, warp % WPR, WPR);
+    d.fetch();
+    pdl_wait();
+    float acc[R] = {};
+    d.run(x, acc);
+    group_sum<R, WPR>(acc, red);
+    if (warp % WPR == 0 && (threadIdx.x & 31) == 0) {
+#pragma unroll
+        for (int r = 0; r < R; ++r)
+            if (g * R + r < rows) y[g * R + r] = acc[r];
+    }
+}
+
+template <class T, int WPR>
+__global__ void __launch_bounds__(GV_WARPS * 32) mingru_step_kernel(const T *__restrict__ w, uint32_t wp, uint32_t ld, const T *x,
+                                                                    const float *__restrict__ zb, const float *__restrict__ xb, float *state, T *out) {
+    __shared__ float red[GV_WARPS][3];
+    pdl_trigger();
+    const int warp = threadIdx.x >> 5;
+    const uint32_t g = blockIdx.x * (GV_WARPS / WPR) + warp / WPR, gi = min(g, wp - 1);
+    RowDot<T, 3, 4> d;
+#pragma unroll
+    for (int r = 0; r < 3; ++r) d.w[r] = w + (size_t)(gi + r * wp) * ld;
+    d.start(ld, warp % WPR, WPR);
+    d.fetch();
+    pdl_wait();
+    float acc[3] = {};
+    d.run(x, acc);
+    group_sum<3, WPR>(acc, red);
+    if (warp % WPR == 0 && (threadIdx.x & 31) == 0 && g < wp) {
+        float z, cand;
+        mingru_gates(acc[0], acc[1], zb[g], xb[g], z, cand);
+        const float s = (1.0f - z) * state[g] + z * cand;
+        state[g] = s;
+        out[g] = Elem<T>::from(s * silu_f32(acc[2]));
+    }
+}
+
+// grid (row groups, picks).  Every CTA repeats the pick from the router logits; CTA 0 of a pick leaves it for the down step.
+template <class T, int WPR>
+__global__ void __launch_bounds__(GV_WARPS * 32) expert_gate_up_kernel(const T *__restrict__ w, uint32_t ff_p, uint32_t ld, const T *x,
+                                                                       const float *logits, RouterRule rule, ExpertAct a, uint32_t *ids,
+                                                                       float *weights, T *act) {
+    __shared__ float red[GV_WARPS][2];
+    __shared__ float probs[MOE_MAX_EXPERTS];
+    __shared__ uint32_t picked[MOE_MAX_USED];
+    __shared__ float wt[MOE_MAX_USED];
+    pdl_trigger();
+    pdl_wait();
+    for (uint32_t e = threadIdx.x; e < rule.n_expert; e += blockDim.x) probs[e] = logits[e];
+    __syncthreads();
+    moe_scores(probs, rule.n_expert, rule.softmax);
+    const int warp = threadIdx.x >> 5;
+    if (warp == 0) moe_pick(probs, nullptr, rule.n_expert, rule.n_used, rule.renorm, picked, wt);
+    __syncthreads();
+    const uint32_t s = blockIdx.y, e = picked[s];
+    if (blockIdx.x == 0 && threadIdx.x == 0) {
+        ids[s] = e;
+        weights[s] = wt[s];
+    }
+    const uint32_t g = blockIdx.x * (GV_WARPS / WPR) + warp / WPR, gi = min(g, ff_p - 1);
+    RowDot<T, 2, 4> d;
+    d.w[0] = w + ((size_t)e * 2 * ff_p + gi) * ld;
+    d.w[1] = d.w[0] + (size_t)ff_p * ld;
+    d.start(ld, warp % WPR, WPR);
+    d.fetch();
+    float acc[2] = {};
+    d.run(x, acc);
+    group_sum<2, WPR>(acc, red);
+    if (warp % WPR == 0 && (threadIdx.x & 31) == 0 && g < ff_p) {
+        const float sc = rule.weight_input ? wt[s] : 1.0f;
+        act[(size_t)s * ff_p + g] = Elem<T>::from(gated_unit(sc * acc[0], sc * acc[1], a));
+    }
+}
+
+template <class T, int WPR>
+__global__ void __launch_bounds__(GV_WARPS * 32) expert_down_kernel(const T *__restrict__ w, uint32_t rows, uint32_t ld, const T *act, uint32_t n_used,
+                                                                    int weight_input, const uint32_t *ids, const float *weights, float *y) {
+    __shared__ float red[GV_WARPS][1];
+    pdl_trigger();
+    pdl_wait();
+    const int warp = threadIdx.x >> 5;
+    const uint32_t g = blockIdx.x * (GV_WARPS / WPR) + warp / WPR, gi = min(g, rows - 1);
+    float total[1] = {0.0f};
+    for (uint32_t s = 0; s < n_used; ++s) {
+        RowDot<T, 1, 8> d;
+        d.w[0] = w + ((size_t)ids[s] * rows + gi) * ld;
+        d.start(ld, warp % WPR, WPR);
+        d.fetch();
+        float acc[1] = {0.0f};
+        d.run(act + (size_t)s * ld, acc);
+        total[0] += weight_input ? acc[0] : weights[s] * acc[0];
+    }
+    group_sum<1, WPR>(total, red);
+    if (warp % WPR == 0 && (threadIdx.x & 31) == 0 && g < rows) y[g] = total[0];
+}
+
+// Warps per row group: enough warps to cover the memory latency when there are few groups.
+int pick_wpr(size_t groups) {
+    const size_t want = (size_t)sm_count() * 14;
+    for (int wpr = 1; wpr < 8; wpr *= 2)
+        if (groups * wpr >= want) return wpr;
+    return 8;
+}
+
+template <class F>
+int32_t with_wpr(int wpr, F f) {
+    switch (wpr) {
+        case 1: return f(std::integral_constant<int, 1>{});
+        case 2: return f(std::integral_constant<int, 2>{});
+        case 4: return f(std::integral_constant<int, 4>{});
+        default: return f(std::integral_constant<int, 8>{});
+    }
+}
+template <class F>
+int32_t with_type(int f32, F f) {
+    return f32 ? f(float{}) : f(bf16{});
+}
+dim3 gv_grid(size_t groups, int wpr, uint32_t y = 1) { return dim3((unsigned)((groups * wpr + GV_WARPS - 1) / GV_WARPS), y); }
+
+}  // namespace
+
+int32_t launch_dense_gemv(const DenseView &w, const void *x, float *y, cudaStream_t st) {
+    const bool two = w.rows >= (uint32_t)sm_count() * 28;
+    const size_t groups = two ? (w.rows + 1) / 2 : w.rows;
+    const int wpr = pick_wpr(groups);
+    count_launch();
+    return with_type(w.f32, [&](auto t) {
+        using T = decltype(t);
+        return with_wpr(wpr, [&](auto n) {
+            constexpr int W = decltype(n)::value;
+            return check_cuda(two ? launch_k(gemv_kernel<T, 2, W>, gv_grid(groups, wpr), dim3(GV_WARPS * 32), 0, st, (const T *)w.w, w.rows, w.ld, (const T *)x, y)
+                                  : launch_k(gemv_kernel<T, 1, W>, gv_grid(groups, wpr), dim3(GV_WARPS * 32), 0, st, (const T *)w.w, w.rows, w.ld, (const T *)x, y),
+                              "dense gemv launch");
+        });
+    });
+}
+
+int32_t launch_mingru_step(const DenseView &w, const void *x, const float *z_bias, const float *x_bias, float *state, void *out, cudaStream_t st) {
+    const uint32_t wp = w.rows / 3;
+    const int wpr = pick_wpr(wp);
+    count_launch();
+    return with_type(w.f32, [&](auto t) {
+        using T = decltype(t);
+        return with_wpr(wpr, [&](auto n) {
+            return check_cuda(launch_k(mingru_step_kernel<T, decltype(n)::value>, gv_grid(wp, wpr), dim3(GV_WARPS * 32), 0, st, (const T *)w.w, wp, w.ld,
+                                       (const T *)x, z_bias, x_bias, state, (T *)out),
+                              "mingru step launch");
+        });
+    });
+}
+
+int32_t launch_expert_gate_up_step(const DenseView &w, const void *x, const float *router_logits, const RouterRule &r, uint32_t ff_p, const ExpertAct &a,
+                                   uint32_t *ids, float *weights, void *act, cudaStream_t st) {
+    const int wpr = pick_wpr((size_t)ff_p * r.n_used);
+    count_launch();
+    return with_type(w.f32, [&](auto t) {
+        using T = decltype(t);
+        return with_wpr(wpr, [&](auto n) {
+            return check_cuda(launch_k(expert_gate_up_kernel<T, decltype(n)::value>, gv_grid(ff_p, wpr, r.n_used), dim3(GV_WARPS * 32), 0, st,
+                                       (const T *)w.w, ff_p, w.ld, (const T *)x, router_logits, r, a, ids, weights, (T *)act),
+                              "expert gate/up launch");
+        });
+    });
+}
+
+int32_t launch_expert_down_step(const DenseView &w, uint32_t rows_per_expert, const void *act, const RouterRule &r, const uint32_t *ids,
+                                const float *weights, float *y, cudaStream_t st) {
+    const int wpr = pick_wpr(rows_per_expert);
+    count_launch();
+    return with_type(w.f32, [&](auto t) {
+        using T = decltype(t);
+        return with_wpr(wpr, [&](auto n) {
+            return check_cuda(launch_k(expert_down_kernel<T, decltype(n)::value>, gv_grid(rows_per_expert, wpr), dim3(GV_WARPS * 32), 0, st,
+                                       (const T *)w.w, rows_per_expert, w.ld, (const T *)act, r.n_used, r.weight_input, ids, weights, y),
+                              "expert down launch");
+        });
+    });
+}
+
+}  // namespace cera

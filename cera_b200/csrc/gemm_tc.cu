@@ -1240,11 +1240,12 @@ int32_t weight_prepare_tc(cera_cuda_weight *w, bool *built) {
     return rc;
 }
 
-uint32_t gemm_tc_status() {
+// bits 8..12: roles of the tcgen05 GEMM
+static const bool g_tc_status_registered = register_kernel_status([] {
     unsigned int v = 0;
     cudaMemcpyFromSymbol(&v, g_tc_status, sizeof(v));
-    return v;
-}
+    return (uint32_t)v << 8;
+});
 
 // One activation matrix against up to three weights (q / k / v, gate / up): the activation operands are converted once
 // and, when every weight has its image, ONE kernel launch covers all of them (the small matrices' CTAs run beside the

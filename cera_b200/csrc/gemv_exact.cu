@@ -630,11 +630,12 @@ int32_t launch_exact_typed(const ExactParams &p0, cudaStream_t st) {
 
 }  // namespace
 
-uint32_t gemv_exact_status() {
+// bit 16: a copy of the reference-order GEMV never arrived
+static const bool g_xg_status_registered = register_kernel_status([] {
     unsigned int v = 0;
     cudaMemcpyFromSymbol(&v, g_xg_status, sizeof(v));
-    return v;
-}
+    return (uint32_t)v << 16;
+});
 
 // CERA_CUDA_GEMV=rows keeps the decode GEMVs on the register-streaming kernel whose f32 order is its own (A/B runs); read once.
 static bool exact_off() {

@@ -334,21 +334,11 @@ int32_t launch_gemv_tma(const GemvSeg *segs, int n_segs, const ActView &x, int e
     return CERA_CUDA_OK;
 }
 
-}  // namespace cera
-
-using namespace cera;
-
-extern "C" {
-
-int32_t cera_cuda_kernel_status(uint32_t *status_out) {
-    if (!status_out) return fail(CERA_CUDA_ERR_BAD_ARG, "kernel_status: null argument");
+// low bits: roles of the TMA-staged GEMV
+static const bool g_tma_status_registered = register_kernel_status([] {
     unsigned int v = 0;
-    CERA_CUDA_TRY(cudaMemcpyFromSymbol(&v, g_tma_status, sizeof(v)));
-    v |= gemm_tc_status() << 8;      // bits 8..12: roles of the tcgen05 GEMM
-    v |= gemv_exact_status() << 16;  // bit 16: a copy of the reference-order GEMV never arrived
-    *status_out = v;
-    if (v) return fail(CERA_CUDA_ERR_TIMEOUT, "a bounded device-side wait ran out (status word %u)", v);
-    return CERA_CUDA_OK;
-}
+    cudaMemcpyFromSymbol(&v, g_tma_status, sizeof(v));
+    return (uint32_t)v;
+});
 
-}  // extern "C"
+}  // namespace cera

@@ -1,0 +1,306 @@
+// Latent attention: keys and values are up-projections of one normed latent per position, so only the latent and one
+// rotated key part per position are cached.  This file: what every path needs (norm, rotation, cache append) and the
+// latent-space form, in which W_uk is applied to the query and W_uv to the weighted sum of latents - the decode step,
+// short prompt portions, and everything in f32.  Scores, softmax and sums are f32.
+#include "dense.cuh"
+#include "tma.cuh"
+
+namespace cera {
+
+namespace {
+
+// One CTA per token.
+template <class T>
+__global__ void __launch_bounds__(256) latent_prepare_kernel(const float *in, LatentShape s, uint32_t start_pos, const uint32_t *pos_dev,
+                                                             const float *__restrict__ c_norm, float eps, const float *__restrict__ rope, T *cache_c,
+                                                             T *cache_r, float *q32, T *qt, float *gate) {
+    __shared__ float red[33];
+    pdl_trigger();
+    pdl_wait();
+    const uint32_t j = blockIdx.x, pos = (pos_dev ? *pos_dev : start_pos) + j, t = threadIdx.x;
+    const float *row = in + (size_t)j * s.in_p, *c = row + s.off_c(), *kr = row + s.off_r(), *gl = row + s.off_g();
+    const float *cs = rope + (size_t)pos * s.rot;  // (cos, sin) of the rot / 2 pairs
+    float ss = 0.0f;
+    for (uint32_t i = t; i < s.rank; i += 256) ss += c[i] * c[i];
+    const float r = 1.0f / sqrtf(cta_sum(ss, red) / (float)s.rank + eps);
+    for (uint32_t i = t; i < s.rank_p; i += 256) cache_c[(size_t)pos * s.rank_p + i] = Elem<T>::from(c[i] * r * c_norm[i]);
+    auto turned = [&](const float *v, uint32_t i) {  // element i of the rotated vector
+        if (i >= s.rot) return 0.0f;
+        const float cv = cs[i & ~1u], sv = cs[i | 1u];
+        return i & 1 ? v[i] * cv + v[i - 1] * sv : v[i] * cv - v[i + 1] * sv;
+    };
+    for (uint32_t i = t; i < s.rot_p; i += 256) cache_r[(size_t)pos * s.rot_p + i] = Elem<T>::from(turned(kr, i));
+    const uint32_t hd = s.dim_p + s.rot_p, total = s.heads * hd;
+    for (uint32_t i = t; i < total; i += 256) {
+        const uint32_t d = i % hd;
+        const float v = d < s.dim_p ? row[i] : turned(row + (i - d) + s.dim_p, d - s.dim_p);
+        if (q32) q32[(size_t)j * total + i] = v;
+        if (qt) qt[(size_t)j * total + i] = Elem<T>::from(v);
+    }
+    for (uint32_t h = t; h < s.heads; h += 256) gate[(size_t)j * s.heads + h] = sigmoid_f32(gl[h]);
+}
+
+// q_lat[j][h] = [W_uk_h^T q_h, rotated part].  grid (64-column slabs of rank_p, heads, queries), 4 x 64 threads: thread
+// (slice of the head's dimensions, column).
+template <class T>
+__global__ void __launch_bounds__(256) latent_query_kernel(const float *q32, LatentShape s, const T *__restrict__ uk, float *q_lat) {
+    __shared__ float part[4][64];
+    pdl_trigger();
+    pdl_wait();
+    const uint32_t h = blockIdx.y, j = blockIdx.z, col = threadIdx.x & 63, sl = threadIdx.x >> 6, c = blockIdx.x * 64 + col;
+    const uint32_t hd = s.dim_p + s.rot_p, ldo = s.rank_p + s.rot_p;
+    const float *q = q32 + ((size_t)j * s.heads + h) * hd;
+    const T *w = uk + (size_t)h * s.dim_p * s.rank_p + c;
+    float acc = 0.0f;
+#pragma unroll 8
+    for (uint32_t d = sl; d < s.dim_p; d += 4) acc = fmaf(q[d], Elem<T>::to(w[(size_t)d * s.rank_p]), acc);
+    part[sl][col] = acc;
+    __syncthreads();
+    float *o = q_lat + ((size_t)j * s.heads + h) * ldo;
+    if (sl == 0) o[c] = part[0][col] + part[1][col] + part[2][col] + part[3][col];
+    if (blockIdx.x == 0)
+        for (uint32_t i = threadIdx.x; i < s.rot_p; i += 256) o[s.rank_p + i] = q[s.dim_p + i];
+}
+
+constexpr int LA_WARPS = 4, LA_KEYS = 32;
+
+// One CTA: (split of the keys, 4 HG heads, query).  Tiles of 32 keys in shared memory; a warp owns HG heads: scores with
+// lane = key, online softmax, weighted latents with lane = columns.
+template <class T, int HG, int NJ>
+__global__ void __launch_bounds__(LA_WARPS * 32) latent_split_kernel(const float *q_lat, LatentShape s, const T *cache_c, const T *cache_r, uint32_t start_pos,
+                                                                     const uint32_t *len_dev, uint32_t splits, int stages, float *part) {
+    constexpr int VN = Elem<T>::N;
+    extern __shared__ __align__(16) uint8_t smem[];
+    pdl_trigger();
+    const uint32_t ql = s.rank_p + s.rot_p, row_b = ql * sizeof(T) + 16, row_v = ql / VN, c_v = s.rank_p / VN;
+    float *qs = reinterpret_cast<float *>(smem);  // [LA_WARPS * HG][ql]
+    uint8_t *tile = smem + (size_t)LA_WARPS * HG * ql * 4;
+    pdl_wait();
+    const uint32_t split = blockIdx.x, h0 = blockIdx.y * LA_WARPS * HG, j = blockIdx.z, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const uint32_t len = len_dev ? *len_dev : start_pos + j + 1;
+    const uint32_t per = ((len + splits - 1) / splits + LA_KEYS - 1) / LA_KEYS * LA_KEYS, k0 = min(split * per, len), k1 = min(k0 + per, len);
+    for (uint32_t i = threadIdx.x; i < LA_WARPS * HG * ql; i += LA_WARPS * 32) {
+        const uint32_t h = h0 + i / ql;
+        qs[i] = h < s.heads ? q_lat[((size_t)j * s.heads + h) * ql + i % ql] : 0.0f;
+    }
+    auto fetch = [&](uint32_t base, int stage) {
+        uint8_t *dst = tile + (size_t)stage * LA_KEYS * row_b;
+        for (uint32_t i = threadIdx.x; i < LA_KEYS * row_v; i += LA_WARPS * 32) {
+            const uint32_t k = i / row_v, v = i - k * row_v;
+            if (base + k < k1) {
+                const T *src = v < c_v ? cache_c + (size_t)(base + k) * s.rank_p + v * VN : cache_r + (size_t)(base + k) * s.rot_p + (v - c_v) * VN;
+                tma::cp_async16(dst + (size_t)k * row_b + v * 16, src);
+            } else {
+                *reinterpret_cast<uint4 *>(dst + (size_t)k * row_b + v * 16) = make_uint4(0, 0, 0, 0);
+            }
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    float m[HG], l[HG], o[HG][NJ * VN];
+#pragma unroll
+    for (int g = 0; g < HG; ++g) {
+        m[g] = -INFINITY;
+        l[g] = 0.0f;
+#pragma unroll
+        for (int i = 0; i < NJ * VN; ++i) o[g][i] = 0.0f;
+    }
+    const float *qw = qs + (size_t)warp * HG * ql;
+    int stage = 0;
+    if (k0 < k1) fetch(k0, 0);
+    for (uint32_t base = k0; base < k1; base += LA_KEYS) {
+        const bool more = base + LA_KEYS < k1 && stages == 2;
+        if (more) fetch(base + LA_KEYS, stage ^ 1);
+        if (more) asm volatile("cp.async.wait_group 1;" ::: "memory");
+        else asm volatile("cp.async.wait_group 0;" ::: "memory");
+        __syncthreads();
+        const uint8_t *tl = tile + (size_t)stage * LA_KEYS * row_b;
+        float sc[HG];
+#pragma unroll
+        for (int g = 0; g < HG; ++g) sc[g] = 0.0f;
+        const uint4 *kv = reinterpret_cast<const uint4 *>(tl + (size_t)lane * row_b);
+        for (uint32_t v = 0; v < row_v; ++v) {
+            float kf[VN];
+            Elem<T>::unpack(kv[v], kf);
+#pragma unroll
+            for (int g = 0; g < HG; ++g) {
+#pragma unroll
+                for (int q4 = 0; q4 < VN / 4; ++q4) {
+                    const float4 q = *reinterpret_cast<const float4 *>(qw + (size_t)g * ql + v * VN + q4 * 4);
+                    sc[g] = fmaf(q.x, kf[q4 * 4], sc[g]);
+                    sc[g] = fmaf(q.y, kf[q4 * 4 + 1], sc[g]);
+                    sc[g] = fmaf(q.z, kf[q4 * 4 + 2], sc[g]);
+                    sc[g] = fmaf(q.w, kf[q4 * 4 + 3], sc[g]);
+                }
+            }
+        }
+#pragma unroll
+        for (int g = 0; g < HG; ++g) {
+            const float v = base + lane < k1 ? sc[g] * s.scale : -INFINITY;
+            const float mn = fmaxf(m[g], warp_max(v));  // (the first key of a tile is always valid: mn is finite)
+            const float alpha = expf(m[g] - mn);
+            sc[g] = expf(v - mn);
+            l[g] = l[g] * alpha + warp_sum(sc[g]);
+            m[g] = mn;
+#pragma unroll
+            for (int i = 0; i < NJ * VN; ++i) o[g][i] *= alpha;
+        }
+        const uint32_t nk = min((uint32_t)LA_KEYS, k1 - base);
+        for (uint32_t k = 0; k < nk; ++k) {
+            float p[HG];
+#pragma unroll
+            for (int g = 0; g < HG; ++g) p[g] = __shfl_sync(0xffffffffu, sc[g], k);
+            const uint4 *cv = reinterpret_cast<const uint4 *>(tl + (size_t)k * row_b);
+#pragma unroll
+            for (int jj = 0; jj < NJ; ++jj) {
+                const uint32_t v = jj * 32 + lane;
+                if (v < c_v) {
+                    float cf[VN];
+                    Elem<T>::unpack(cv[v], cf);
+#pragma unroll
+                    for (int g = 0; g < HG; ++g)
+#pragma unroll
+                        for (int i = 0; i < VN; ++i) o[g][jj * VN + i] = fmaf(p[g], cf[i], o[g][jj * VN + i]);
+                }
+            }
+        }
+        __syncthreads();
+        if (stages == 2) stage ^= 1;
+        else if (base + LA_KEYS < k1) fetch(base + LA_KEYS, 0);
+    }
+#pragma unroll
+    for (int g = 0; g < HG; ++g) {
+        const uint32_t h = h0 + warp * HG + g;
+        if (h >= s.heads) continue;
+        float *po = part + (((size_t)j * s.heads + h) * splits + split) * (s.rank_p + 2);
+        if (lane == 0) {
+            po[0] = m[g];
+            po[1] = l[g];
+        }
+#pragma unroll
+        for (int jj = 0; jj < NJ; ++jj)
+            if (jj * 32 + lane < c_v) {
+#pragma unroll
+                for (int i = 0; i < VN; ++i) po[2 + (jj * 32 + lane) * VN + i] = o[g][jj * VN + i];
+            }
+    }
+}
+
+// grid (slabs of a head's value rows, heads, queries): combine the splits with the sink, then this slab's rows of W_uv.
+template <class T>
+__global__ void __launch_bounds__(256) latent_merge_kernel(const float *part, LatentShape s, uint32_t splits, const float *__restrict__ sink,
+                                                           const float *gate, const T *__restrict__ uv, T *out, size_t ldo) {
+    extern __shared__ __align__(16) float lat[];  // [rank_p]
+    __shared__ float wt[LATENT_MAX_SPLITS];
+    pdl_trigger();
+    pdl_wait();
+    const uint32_t h = blockIdx.y, j = blockIdx.z, ps = s.rank_p + 2, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const float *p = part + ((size_t)j * s.heads + h) * splits * ps;
+    if (warp == 0) {
+        const float sk = sink[h];
+        float mx = sk;
+        for (uint32_t i = lane; i < splits; i += 32) mx = fmaxf(mx, p[(size_t)i * ps]);
+        mx = warp_max(mx);
+        float den = 0.0f;
+        for (uint32_t i = lane; i < splits; i += 32) {
+            const float e = expf(p[(size_t)i * ps] - mx);
+            wt[i] = e;
+            den += e * p[(size_t)i * ps + 1];
+        }
+        den = warp_sum(den) + expf(sk - mx);
+        __syncwarp();
+        for (uint32_t i = lane; i < splits; i += 32) wt[i] /= den;
+    }
+    __syncthreads();
+    for (uint32_t c = threadIdx.x; c < s.rank_p; c += 256) {
+        float v = 0.0f;
+        for (uint32_t i = 0; i < splits; ++i) v = fmaf(wt[i], p[(size_t)i * ps + 2 + c], v);
+        lat[c] = v;
+    }
+    __syncthreads();
+    const float gt = gate[(size_t)j * s.heads + h];
+    const uint32_t slab = (s.vdim_p + gridDim.x - 1) / gridDim.x, v0 = blockIdx.x * slab, v1 = min(v0 + slab, s.vdim_p);
+    for (uint32_t v = v0 + warp; v < v1; v += 8) {
+        const uint4 *w = reinterpret_cast<const uint4 *>(uv + ((size_t)h * s.vdim_p + v) * s.rank_p);
+        float acc = 0.0f;
+        for (uint32_t c = lane; c < s.rank_p / Elem<T>::N; c += 32) {
+            float wf[Elem<T>::N];
+            Elem<T>::unpack(w[c], wf);
+#pragma unroll
+            for (int i = 0; i < Elem<T>::N; ++i) acc = fmaf(wf[i], lat[c * Elem<T>::N + i], acc);
+        }
+        acc = warp_sum(acc);
+        if (lane == 0) out[j * ldo + (size_t)h * s.vdim_p + v] = Elem<T>::from(acc * gt);
+    }
+}
+
+template <class T, int HG, int NJ>
+int32_t launch_split(const LatentScratch &ws, const LatentShape &s, const void *cc, const void *cr, size_t n, size_t start_pos, const uint32_t *len_dev,
+                     uint32_t splits, cudaStream_t st) {
+    const uint32_t ql = s.rank_p + s.rot_p;
+    const size_t qb = (size_t)LA_WARPS * HG * ql * 4, tb = (size_t)LA_KEYS * (ql * sizeof(T) + 16);
+    const int stages = qb + 2 * tb <= 220 * 1024 ? 2 : 1;
+    const size_t smem = qb + stages * tb;
+    if (smem > 220 * 1024) return fail(CERA_CUDA_ERR_UNSUPPORTED, "latent attention: rank %u with %u rotated dimensions", s.rank, s.rot);
+    auto k = latent_split_kernel<T, HG, NJ>;
+    CERA_CUDA_TRY(cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024));
+    count_launch();
+    return check_cuda(launch_k(k, dim3(splits, (s.heads + LA_WARPS * HG - 1) / (LA_WARPS * HG), (unsigned)n), dim3(LA_WARPS * 32), smem, st, (const float *)ws.q_lat,
+                               s, (const T *)cc, (const T *)cr, (uint32_t)start_pos, len_dev, splits, stages, ws.part),
+                      "latent split launch");
+}
+
+template <class T>
+int32_t latent_attention(const float *q32, const LatentShape &s, const void *uk, const void *uv, const void *cc, const void *cr, const float *sink,
+                         const float *gate, size_t n, size_t start_pos, const uint32_t *len_dev, uint32_t splits, const LatentScratch &ws, void *out,
+                         size_t ldo, cudaStream_t st) {
+    count_launch();
+    CERA_CUDA_TRY(launch_k(latent_query_kernel<T>, dim3(s.rank_p / 64, s.heads, (unsigned)n), dim3(256), 0, st, q32, s, (const T *)uk, ws.q_lat));
+    const uint32_t nj = (s.rank_p / Elem<T>::N + 31) / 32;
+    const bool few = s.heads <= 8;  // one head per warp
+    auto split = [&](auto hg) -> int32_t {
+        constexpr int HG = decltype(hg)::value;
+        if (nj <= 1) return launch_split<T, HG, 1>(ws, s, cc, cr, n, start_pos, len_dev, splits, st);
+        if (nj <= 2) return launch_split<T, HG, 2>(ws, s, cc, cr, n, start_pos, len_dev, splits, st);
+        if (nj <= 4) return launch_split<T, HG, 4>(ws, s, cc, cr, n, start_pos, len_dev, splits, st);
+        if constexpr (Elem<T>::N == 4)
+            if (nj <= 8) return launch_split<T, HG, 8>(ws, s, cc, cr, n, start_pos, len_dev, splits, st);
+        return fail(CERA_CUDA_ERR_UNSUPPORTED, "latent attention: rank %u", s.rank);
+    };
+    CERA_TRY(few ? split(std::integral_constant<int, 1>{}) : split(std::integral_constant<int, 4>{}));
+    const uint32_t slabs = n == 1 ? 4 : 1;
+    count_launch();
+    return check_cuda(launch_k(latent_merge_kernel<T>, dim3(slabs, s.heads, (unsigned)n), dim3(256), (size_t)s.rank_p * 4, st, (const float *)ws.part, s, splits,
+                               sink, gate, (const T *)uv, (T *)out, ldo),
+                      "latent merge launch");
+}
+
+}  // namespace
+
+uint32_t latent_splits(size_t n_positions) {
+    uint32_t s = 1;
+    while (s < LATENT_MAX_SPLITS && s * 64 < n_positions) s *= 2;
+    return s;
+}
+
+int32_t launch_latent_prepare(const float *in, const LatentShape &s, size_t n, size_t start_pos, const uint32_t *pos_dev, const float *c_norm, float eps,
+                              const float *rope_table, void *cache_c, void *cache_r, int f32, float *q32, void *qt, float *gate, cudaStream_t st) {
+    if (n == 0) return CERA_CUDA_OK;
+    count_launch();
+    if (f32)
+        return check_cuda(launch_k(latent_prepare_kernel<float>, dim3((unsigned)n), dim3(256), 0, st, in, s, (uint32_t)start_pos, pos_dev, c_norm, eps,
+                                   rope_table, (float *)cache_c, (float *)cache_r, q32, (float *)qt, gate), "latent prepare launch");
+    return check_cuda(launch_k(latent_prepare_kernel<bf16>, dim3((unsigned)n), dim3(256), 0, st, in, s, (uint32_t)start_pos, pos_dev, c_norm, eps, rope_table,
+                               (bf16 *)cache_c, (bf16 *)cache_r, q32, (bf16 *)qt, gate), "latent prepare launch");
+}
+
+int32_t launch_latent_attention(const float *q32, const LatentShape &s, const DenseView &uk, const DenseView &uv, const void *cache_c, const void *cache_r,
+                                const float *sink, const float *gate, size_t n, size_t start_pos, const uint32_t *len_dev, uint32_t splits,
+                                const LatentScratch &ws, void *out, size_t ldo, cudaStream_t st) {
+    if (n == 0) return CERA_CUDA_OK;
+    if (splits == 0 || splits > LATENT_MAX_SPLITS || n * splits > LATENT_MAX_SPLITS)
+        return fail(CERA_CUDA_ERR_BAD_ARG, "latent attention: %zu queries x %u splits", n, splits);
+    return uk.f32 ? latent_attention<float>(q32, s, uk.w, uv.w, cache_c, cache_r, sink, gate, n, start_pos, len_dev, splits, ws, out, ldo, st)
+                  : latent_attention<bf16>(q32, s, uk.w, uv.w, cache_c, cache_r, sink, gate, n, start_pos, len_dev, splits, ws, out, ldo, st);
+}
+
+}  // namespace cera

@@ -32,6 +32,7 @@
 #include <new>
 
 #include "gemv_item.cuh"
+#include "moe_route.cuh"
 #include "ops.h"
 #include "weight.h"
 
@@ -39,101 +40,10 @@ using namespace cera;
 
 namespace {
 
-constexpr int MOE_MAX_EXPERTS = 256;  // the reference's stack buffer (lfm2.rs:180)
-constexpr int MOE_MAX_USED = 16;
 constexpr int MOE_NC = 8;             // token columns per work item
 constexpr int MOE_WARPS = 8;
 
 constexpr int MOE_NC_MMA = 64;        // ... when the projections run on the tensor-core GEMM
-
-// ---- routing -------------------------------------------------------------------------------------
-// One CTA per token.  Warps take experts round-robin; lane-strided f32 dot, shuffle tree.
-__global__ void __launch_bounds__(256) moe_route_kernel(const float *__restrict__ x, const float *__restrict__ router,
-                                                        const float *__restrict__ bias, uint32_t hidden, uint32_t n_expert,
-                                                        uint32_t n_used, int softmax_gate, uint32_t *ids, float *weights,
-                                                        uint32_t *counts) {
-    __shared__ float probs[MOE_MAX_EXPERTS];
-    const uint32_t j = blockIdx.x;
-    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    const float *xj = x + (size_t)j * hidden;
-    for (uint32_t e = warp; e < n_expert; e += blockDim.x >> 5) {
-        const float *r = router + (size_t)e * hidden;
-        float acc = 0.0f;
-        for (uint32_t i = lane; i < hidden; i += 32) acc = fmaf(r[i], xj[i], acc);
-        acc = warp_sum(acc);
-        if (lane == 0) probs[e] = acc;
-    }
-    __syncthreads();
-    if (threadIdx.x != 0) return;
-    if (softmax_gate) {
-        float mx = probs[0];
-        for (uint32_t e = 1; e < n_expert; ++e) mx = fmaxf(mx, probs[e]);
-        float sum = 0.0f;
-        for (uint32_t e = 0; e < n_expert; ++e) {
-            probs[e] = expf(probs[e] - mx);
-            sum += probs[e];
-        }
-        for (uint32_t e = 0; e < n_expert; ++e) probs[e] = probs[e] / sum;
-    } else {
-        for (uint32_t e = 0; e < n_expert; ++e) probs[e] = 1.0f / (1.0f + expf(-probs[e]));
-    }
-    uint32_t picked[MOE_MAX_USED];
-    float w[MOE_MAX_USED];
-    float denom = 0.0f;
-    for (uint32_t s = 0; s < n_used; ++s) {
-        int best = -1;
-        float best_v = 0.0f;
-        for (uint32_t e = 0; e < n_expert; ++e) {
-            bool taken = false;
-            for (uint32_t t = 0; t < s; ++t) taken |= picked[t] == e;
-            if (taken) continue;
-            const float v = probs[e] + (bias ? bias[e] : 0.0f);
-            // total order on finite values; strict > keeps the lower index on ties
-            if (best < 0 || v > best_v) {
-                best = (int)e;
-                best_v = v;
-            }
-        }
-        picked[s] = (uint32_t)best;
-        w[s] = probs[best];
-        denom += w[s];
-    }
-    denom = fmaxf(denom, 1.0f / 16384.0f);
-    for (uint32_t s = 0; s < n_used; ++s) {
-        ids[(size_t)j * n_used + s] = picked[s];
-        weights[(size_t)j * n_used + s] = w[s] / denom;
-        atomicAdd(counts + picked[s], 1u);
-    }
-}
-
-// Appends the work items of one expert's `c` entries starting at bucket offset `off`: items of `nc` columns go to
-// the main list; a last item of at most `small_nc` columns (0 = no such list) goes to the list of narrow items at
-// tiles[cap...], which a narrower kernel serves.
-__device__ __forceinline__ void moe_emit_items(MoeTile *tiles, uint32_t cap, uint32_t &t, uint32_t &ts, uint32_t e, uint32_t off,
-                                               uint32_t c, uint32_t nc, uint32_t small_nc) {
-    for (uint32_t f = 0; f < c; f += nc) {
-        const uint32_t n = c - f < nc ? c - f : nc;
-        if (small_nc && n <= small_nc) tiles[cap + ts++] = MoeTile{e, off + f, n};
-        else tiles[t++] = MoeTile{e, off + f, n};
-    }
-}
-
-// One CTA: bucket offsets, cursors, and the work lists (n_tiles[0] main, n_tiles[1] narrow).  counts is zeroed again
-// for the next call.
-__global__ void moe_plan_kernel(uint32_t *counts, uint32_t n_expert, uint32_t nc, uint32_t small_nc, uint32_t cap, uint32_t *cursor,
-                                MoeTile *tiles, uint32_t *n_tiles) {
-    if (threadIdx.x != 0) return;
-    uint32_t off = 0, t = 0, ts = 0;
-    for (uint32_t e = 0; e < n_expert; ++e) {
-        const uint32_t c = counts[e];
-        cursor[e] = off;
-        moe_emit_items(tiles, cap, t, ts, e, off, c, nc, small_nc);
-        off += c;
-        counts[e] = 0;
-    }
-    n_tiles[0] = t;
-    n_tiles[1] = ts;
-}
 
 // One CTA per (token, pick): take the next place in the expert's bucket and copy the token's Q8_0 column there.
 __global__ void __launch_bounds__(128) moe_scatter_kernel(const uint32_t *__restrict__ ids, uint32_t n_used, uint32_t hidden,
@@ -540,8 +450,7 @@ int32_t moe_ffn_ep(cera_cuda_moe *h, const float *x_dev, size_t n, int32_t softm
     CERA_TRY(launch_tp_tick(h->ep_words, st));
     if (n) {
         CERA_TRY(launch_quantize(x_dev, hs, n, false, h->xs, h->xq, h->xsum, st));
-        moe_route_kernel<<<(unsigned)n, 256, 0, st>>>(x_dev, h->router, h->bias, hs, E, ku, softmax_gate, h->ids, h->weights, counts_mine);
-        count_launch();
+        CERA_TRY(launch_moe_route(x_dev, hs, n, h->router, h->bias, hs, E, ku, softmax_gate, 1, h->ids, h->weights, counts_mine, st));
     }
     // all ranks learn all counts
     const TpRange cr{(uint32_t)((char *)counts_mine - h->region), E * 4};
@@ -682,13 +591,12 @@ int32_t cera_cuda_moe_ffn(cera_cuda_moe *h, const float *x_dev, size_t n, int32_
     const uint32_t nc = single ? 1 : mma ? MOE_NC_MMA : MOE_NC;
     const uint32_t max_tiles = (uint32_t)(entries / nc + (single ? 0 : h->n_expert));
     CERA_TRY(launch_quantize(x_dev, hs, n, false, h->xs, h->xq, h->xsum, st));
-    moe_route_kernel<<<(unsigned)n, 256, 0, st>>>(x_dev, h->router, h->bias, hs, h->n_expert, ku, softmax_gate, h->ids, h->weights,
-                                                  h->counts);
+    CERA_TRY(launch_moe_route(x_dev, hs, n, h->router, h->bias, hs, h->n_expert, ku, softmax_gate, 1, h->ids, h->weights, h->counts, st));
     const uint32_t cap = (uint32_t)(h->max_total * ku + h->n_expert), max_small = h->n_expert;
-    moe_plan_kernel<<<1, 32, 0, st>>>(h->counts, h->n_expert, nc, mma ? nc / 2 : 0, cap, h->cursor, h->tiles, h->n_tiles);
+    CERA_TRY(launch_moe_plan(h->counts, h->n_expert, nc, mma ? nc / 2 : 0, cap, h->cursor, h->tiles, h->n_tiles, st));
     moe_scatter_kernel<<<(unsigned)entries, 128, 0, st>>>(h->ids, ku, hs, ActView{h->xs, h->xq, h->xsum}, h->cursor, h->entry_of,
                                                           h->g_scales, h->g_quants, h->g_sums);
-    count_launch(3);
+    count_launch();
     CERA_CUDA_TRY(cudaGetLastError());
     MoeGemmParams p{};
     p.w[0] = h->gate->v;

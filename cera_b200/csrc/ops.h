@@ -81,13 +81,17 @@ struct GemmTarget {
 };
 int32_t launch_gemm_tc_multi(const GemmTarget *t, int count, const ActView &x, size_t n, size_t ldy, int epilogue, cudaStream_t st,
                              bool *taken);
-uint32_t gemm_tc_status();  // nonzero after a bounded wait of that kernel ran out
-uint32_t gemv_exact_status();
 // One work item of an expert-grouped GEMM: `count` consecutive activation columns starting at `first` go through
 // expert `expert`'s rows of a stacked weight matrix (built on the device by the routed-FFN kernels).
 struct MoeTile {
     uint32_t expert, first, count;
 };
+// Routing of a batch (moe_route.cu): x rows of ld_x floats; counts[e] += entries of expert e; and the work lists over the
+// buckets (counts is zeroed, n_tiles[0] main list, n_tiles[1] the list of items of at most small_nc columns at tiles + cap).
+int32_t launch_moe_route(const float *x, size_t ld_x, size_t n, const float *router, const float *bias, uint32_t hidden, uint32_t n_expert,
+                         uint32_t n_used, int softmax_gate, int renorm, uint32_t *ids, float *weights, uint32_t *counts, cudaStream_t st);
+int32_t launch_moe_plan(uint32_t *counts, uint32_t n_expert, uint32_t nc, uint32_t small_nc, uint32_t cap, uint32_t *cursor, MoeTile *tiles,
+                        uint32_t *n_tiles, cudaStream_t st);
 // The tensor-core GEMM over a device-side list of such items (one column tile of up to `bn` = 64 or 32 columns per item):
 // w stacks `rows_per_expert` rows per expert; cell (row i of the expert, column c) goes to out[c * ldc + i].
 // *taken = false: no tensor-core path for this weight type / shape.

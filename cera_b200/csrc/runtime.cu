@@ -26,6 +26,15 @@ int32_t check_cuda(cudaError_t e, const char *what) {
     return fail(code, "%s: %s", what, cudaGetErrorString(e));
 }
 
+static uint32_t (*g_status_readers[16])();
+static int g_n_status_readers = 0;
+
+bool register_kernel_status(uint32_t (*reader)()) {
+    if (g_n_status_readers >= 16) return false;
+    g_status_readers[g_n_status_readers++] = reader;
+    return true;
+}
+
 void count_launch(int n) { g_launches.fetch_add((uint64_t)n, std::memory_order_relaxed); }
 uint64_t launches_so_far() { return g_launches.load(std::memory_order_relaxed); }
 
@@ -55,6 +64,16 @@ int sm_count() {
 extern "C" {
 
 const char *cera_cuda_last_error(void) { return cera::g_err; }
+
+int32_t cera_cuda_kernel_status(uint32_t *status_out) {
+    if (!status_out) return cera::fail(CERA_CUDA_ERR_BAD_ARG, "kernel_status: null argument");
+    uint32_t v = 0;
+    for (int i = 0; i < cera::g_n_status_readers; ++i) v |= cera::g_status_readers[i]();
+    CERA_CUDA_TRY(cudaGetLastError());
+    *status_out = v;
+    if (v) return cera::fail(CERA_CUDA_ERR_TIMEOUT, "a bounded device-side wait ran out (status word %u)", v);
+    return CERA_CUDA_OK;
+}
 
 int32_t cera_cuda_device_count(int32_t *count) {
     if (!count) return cera::fail(CERA_CUDA_ERR_BAD_ARG, "count is null");

@@ -22,6 +22,29 @@ class Role(enum.IntEnum):
     FFN_UP = 10
     FFN_DOWN = 11
     ROPE_FREQS = 12
+    # models described layer by layer (layered.py)
+    BIGRAM_EMBD = 13
+    MIX_PRE_NORM = 14
+    MIX_POST_NORM = 15
+    FF_PRE_NORM = 16
+    FF_POST_NORM = 17
+    MIX_OUTPUT = 18
+    LATENT_Q = 20
+    LATENT_DOWN = 21
+    LATENT_NORM = 22
+    LATENT_UP_K = 23
+    LATENT_UP_V = 24
+    LATENT_SINK = 25
+    LATENT_GATE = 26
+    GRU_Z = 30
+    GRU_Z_BIAS = 31
+    GRU_X = 32
+    GRU_X_BIAS = 33
+    GRU_GATE = 34
+    ROUTER = 40
+    EXPERT_GATE = 41
+    EXPERT_UP = 42
+    EXPERT_DOWN = 43
 
 
 ModelConfig = Config
@@ -56,16 +79,21 @@ class CudaModel:
 
     def add_tensor(self, role, layer, ggml_type, rows, cols, data):
         """data: numpy array / bytes (host) or a torch CUDA tensor (device) of raw GGUF bytes."""
+        ptr, nbytes, keep = self._raw(data)
+        check(lib.cera_cuda_model_add_tensor(self.handle, int(role), layer, ggml_type, rows, cols, C.c_void_p(ptr),
+                                             nbytes))
+        del keep
+
+    @staticmethod
+    def _raw(data):
+        """(address, bytes, the object that owns them)."""
         if isinstance(data, (bytes, bytearray)):
             data = np.frombuffer(data, dtype=np.uint8)
         if isinstance(data, np.ndarray):
             data = np.ascontiguousarray(data)
-            ptr, nbytes = data.ctypes.data, data.nbytes
-        else:
-            data = data.contiguous()
-            ptr, nbytes = data.data_ptr(), data.numel() * data.element_size()
-        check(lib.cera_cuda_model_add_tensor(self.handle, int(role), layer, ggml_type, rows, cols, C.c_void_p(ptr),
-                                             nbytes))
+            return data.ctypes.data, data.nbytes, data
+        data = data.contiguous()
+        return data.data_ptr(), data.numel() * data.element_size(), data
 
     def finalize(self):
         check(lib.cera_cuda_model_finalize(self.handle))
@@ -102,6 +130,19 @@ class CudaModel:
         check(lib.cera_cuda_forward_prefill_logits_all(self.handle, tokens.ctypes.data_as(C.c_void_p), tokens.size, start_pos,
                                                        out.ctypes.data_as(C.c_void_p)))
         return out
+
+    def forward_prefill_logits_at(self, tokens, start_pos, want):
+        """Logits of chosen places of a prompt portion -> float32 [len(want), vocab]; an empty list only extends the state."""
+        tokens = np.ascontiguousarray(tokens, dtype=np.uint32)
+        want = np.ascontiguousarray(want, dtype=np.uint32)
+        order, back = np.unique(want, return_inverse=True)  # the library takes ascending places
+        out = np.empty((order.size, self.cfg.vocab_size), dtype=np.float32)
+        order = np.ascontiguousarray(order, dtype=np.uint32)
+        pad = np.zeros(1, dtype=np.uint32)
+        check(lib.cera_cuda_forward_prefill_logits_at(self.handle, tokens.ctypes.data_as(C.c_void_p), tokens.size, start_pos,
+                                                      (order if order.size else pad).ctypes.data_as(C.c_void_p), order.size,
+                                                      out.ctypes.data_as(C.c_void_p)))
+        return out[back.reshape(-1)]
 
     def truncate_kv(self, n):
         check(lib.cera_cuda_truncate_kv(self.handle, n))

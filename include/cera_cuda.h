@@ -258,8 +258,66 @@ enum {
     CERA_ROLE_FFN_GATE = 9,
     CERA_ROLE_FFN_UP = 10,
     CERA_ROLE_FFN_DOWN = 11,
-    CERA_ROLE_ROPE_FREQS = 12 /* rope_freqs.weight (F32, optional) */
+    CERA_ROLE_ROPE_FREQS = 12, /* rope_freqs.weight (F32, optional) */
+    /* Models described layer by layer (cera_cuda_model_create_layered); TOKEN_EMBD, OUTPUT_NORM and OUTPUT as above. */
+    CERA_ROLE_BIGRAM_EMBD = 13,    /* [buckets + 1][hidden] */
+    CERA_ROLE_MIX_PRE_NORM = 14,   /* norm before a layer's mixer: one number or hidden_size numbers */
+    CERA_ROLE_MIX_POST_NORM = 15,  /* norm of the mixer's output, before the residual sum */
+    CERA_ROLE_FF_PRE_NORM = 16,
+    CERA_ROLE_FF_POST_NORM = 17,
+    CERA_ROLE_MIX_OUTPUT = 18,     /* output projection of any mixer */
+    CERA_ROLE_LATENT_Q = 20,       /* [heads * (head_dim + rot_dim)][hidden], per head unrotated then rotated rows */
+    CERA_ROLE_LATENT_DOWN = 21,    /* [kv_rank + rot_dim][hidden] */
+    CERA_ROLE_LATENT_NORM = 22,    /* [kv_rank] */
+    CERA_ROLE_LATENT_UP_K = 23,    /* [heads * head_dim][kv_rank] */
+    CERA_ROLE_LATENT_UP_V = 24,    /* [heads * value_dim][kv_rank] */
+    CERA_ROLE_LATENT_SINK = 25,    /* [heads] */
+    CERA_ROLE_LATENT_GATE = 26,    /* [heads][hidden] */
+    CERA_ROLE_GRU_Z = 30,          /* [recurrent_width][hidden] */
+    CERA_ROLE_GRU_Z_BIAS = 31,
+    CERA_ROLE_GRU_X = 32,
+    CERA_ROLE_GRU_X_BIAS = 33,
+    CERA_ROLE_GRU_GATE = 34,
+    CERA_ROLE_ROUTER = 40,         /* [experts][hidden] */
+    CERA_ROLE_EXPERT_GATE = 41,    /* one expert's [ff_width][hidden] (cera_cuda_model_add_expert_tensor) */
+    CERA_ROLE_EXPERT_UP = 42,
+    CERA_ROLE_EXPERT_DOWN = 43     /* [hidden][ff_width] */
 };
+
+/* A decoder described layer by layer: each layer names its token mixer and its feed-forward with their sizes and
+ * constants.  Weights are dense (bf16 or f32).  No counterpart in the reference. */
+enum { CERA_MIXER_LATENT_ATTENTION = 1, CERA_MIXER_MINGRU = 2 };
+enum { CERA_FF_NONE = 0, CERA_FF_MOE = 1 };
+typedef struct {
+    int32_t mixer;
+    int32_t ff;
+    /* latent attention: per head head_dim unrotated and rot_dim rotated query / key dimensions; keys and values are
+     * up-projections of one normed latent of kv_rank numbers per position, the rotated key part is shared by all heads.
+     * Adjacent dimensions rotate in pairs by pos * rope_base^(-2i / rot_dim).  The softmax denominator also holds
+     * exp(sink) per head; each head's output is multiplied by sigmoid(gate). */
+    uint32_t n_heads, head_dim, rot_dim, value_dim, kv_rank;
+    float rope_base, attn_scale;
+    /* gated recurrence: S = (1 - z) S + z candidate, per element, recurrent_width elements */
+    uint32_t recurrent_width;
+    /* routed feed-forward of n_experts gated units, n_used per token.  Unit: g = min(gate, limit), u = clamp(up, +-limit),
+     * y = g * sigmoid(act_alpha g) * (u + act_shift), then the down projection.  router_softmax: scores are a softmax
+     * instead of a sigmoid; router_renorm: the chosen scores are divided by their sum; the scores multiply the unit's
+     * input (weight_input != 0) or its output. */
+    uint32_t ff_width, n_experts, n_used;
+    float act_limit, act_alpha, act_shift;
+    int32_t router_softmax, router_renorm, weight_input;
+} cera_cuda_layer_desc;
+
+typedef struct {
+    uint32_t n_layers, hidden_size, vocab_size, max_seq_len;
+    float norm_eps;
+    int32_t dtype;  /* CERA_TYPE_BF16: bf16 matrix products and activations; CERA_TYPE_F32: everything in f32 */
+    int32_t device;
+    /* bigram embedding: row (previous * mul_prev + token * mul_cur) mod buckets, row `buckets` for the first token;
+     * buckets == 0: none */
+    uint32_t bigram_buckets;
+    uint64_t bigram_mul_prev, bigram_mul_cur;
+} cera_cuda_layered_config;
 
 CERA_API int32_t cera_cuda_model_create(const cera_cuda_config *cfg, cera_cuda_model **out);
 /* Tensor parallelism over output rows, the axis the reference itself parallelises
@@ -278,6 +336,14 @@ CERA_API int32_t cera_cuda_model_set_tp(cera_cuda_model *m, uint32_t rank, uint3
 CERA_API int32_t cera_cuda_model_add_tensor(cera_cuda_model *m, int32_t role, int32_t layer,
                                             int32_t ggml_type, size_t rows, size_t cols,
                                             const void *bytes, size_t nbytes);
+/* The same model object for a decoder described layer by layer; layers[cfg->n_layers].  Every model-level call below
+ * works on it except those that name dense tensors or parallelism (set_tp, tp_*, attach_lora, kv_shift, *_layer):
+ * CERA_CUDA_ERR_UNSUPPORTED.  Tensors come as BF16, F16 or F32 and are converted to cfg->dtype. */
+CERA_API int32_t cera_cuda_model_create_layered(const cera_cuda_layered_config *cfg, const cera_cuda_layer_desc *layers,
+                                                cera_cuda_model **out);
+/* One expert's matrix of a routed feed-forward. */
+CERA_API int32_t cera_cuda_model_add_expert_tensor(cera_cuda_model *m, int32_t role, int32_t layer, int32_t expert, int32_t type,
+                                                   size_t rows, size_t cols, const void *bytes, size_t nbytes);
 /* Checks every required tensor is present, allocates KV and scratch, and
  * records the decode step.  Must precede the first forward. */
 CERA_API int32_t cera_cuda_model_finalize(cera_cuda_model *m);
@@ -312,7 +378,8 @@ CERA_API int32_t cera_cuda_generate_greedy(cera_cuda_model *m, uint32_t first_to
  * equal seq_len; logits of the last token (may be NULL). */
 CERA_API int32_t cera_cuda_forward_prefill(cera_cuda_model *m, const uint32_t *tokens, size_t n,
                                            size_t start_pos, float *logits_out);
-/* Model::truncate_kv (mod.rs:251-283). */
+/* Model::truncate_kv (mod.rs:251-283).  A model with recurrent layers can only be truncated to 0 (a new sequence):
+ * its state at an earlier position is gone, CERA_CUDA_ERR_UNSUPPORTED.  Take a snapshot to come back. */
 CERA_API int32_t cera_cuda_truncate_kv(cera_cuda_model *m, size_t len);
 /* LoRA adapters (cera/src/lora.rs; the reference carries them on InferenceState::lora and applies
  * them in forward_attn_block / forward_ffn_block, cera/src/model/transformer.rs:1383-1387, 1519-1528,
@@ -331,6 +398,10 @@ CERA_API int32_t cera_cuda_model_detach_lora(cera_cuda_model *m);
  * on the host, token-major. */
 CERA_API int32_t cera_cuda_forward_prefill_logits_all(cera_cuda_model *m, const uint32_t *tokens, size_t n,
                                                       size_t start_pos, float *logits_out);
+/* The same for chosen positions of the portion: want[n_want] ascending places among the n tokens (NULL: all of them),
+ * logits_out[n_want][vocab].  n_want == 0 only extends the state. */
+CERA_API int32_t cera_cuda_forward_prefill_logits_at(cera_cuda_model *m, const uint32_t *tokens, size_t n, size_t start_pos,
+                                                     const uint32_t *want, size_t n_want, float *logits_out);
 /* Model::shift_kv (cera/src/model/llama.rs:1728-1738 -> InferenceState::shift_kv_with_rope,
  * cera/src/kv_cache.rs:1091-1320): drop cached positions [n_keep, n_keep + shift), move the rest down
  * and rotate every moved K head by R(-shift) with the model's RoPE layout and frequency factors; V
