@@ -99,12 +99,17 @@ struct DenseGemm {
     // columns [first, first + count)
     const MoeTile *tiles = nullptr;
     const uint32_t *n_tiles = nullptr;
-    uint32_t max_tiles = 0, rows_per_expert = 0;
+    uint32_t max_tiles = 0, rows_per_expert = 0, group_columns = 0;  // group_columns: most columns of an item
     // DENSE_GATED_UNIT (grouped): rows_per_expert = 2 ff_p, out [columns][ff_p] of T = unit(scale * gate, scale * up)
     ExpertAct act;
     const float *col_scale = nullptr;
 };
-constexpr uint32_t DENSE_GROUP_COLUMNS = 128;  // columns of a grouped item
+// Columns of a grouped item when `entries` columns spread over n_expert experts.
+constexpr uint32_t DENSE_GROUP_MIN = 32;
+inline uint32_t dense_group_columns(uint32_t entries, uint32_t n_expert) {
+    const uint32_t avg = entries / n_expert;
+    return avg <= 24 ? 32 : avg <= 48 ? 64 : 128;
+}
 int32_t launch_dense_gemm(const DenseGemm &g, cudaStream_t st);
 // The bf16 product on tcgen05 / TMEM.  *taken = false: not its case, nothing launched.
 int32_t launch_dense_gemm_tc(const DenseGemm &g, cudaStream_t st, bool *taken);

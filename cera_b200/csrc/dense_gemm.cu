@@ -15,7 +15,7 @@ __global__ void __launch_bounds__(256) dense_gemm_kernel(DenseGemm g) {
     pdl_wait();
     uint32_t row_base = 0, rows = g.w.rows, first = blockIdx.y * GM_TILE, end = g.n;
     if (g.tiles) {  // blockIdx.y walks (item, 64-column part)
-        const uint32_t parts = DENSE_GROUP_COLUMNS / GM_TILE, item = blockIdx.y / parts;
+        const uint32_t parts = (g.group_columns + GM_TILE - 1) / GM_TILE, item = blockIdx.y / parts;
         if (item >= *g.n_tiles) return;
         const MoeTile t = g.tiles[item];
         row_base = t.expert * g.rows_per_expert;
@@ -102,7 +102,7 @@ int32_t launch_dense_gemm(const DenseGemm &g, cudaStream_t st) {
         return check_cuda(e, "cudaFreeAsync(gated unit)");
     }
     const uint32_t rows = g.tiles ? g.rows_per_expert : g.w.rows;
-    const dim3 grid((rows + GM_TILE - 1) / GM_TILE, g.tiles ? g.max_tiles * (DENSE_GROUP_COLUMNS / GM_TILE) : (g.n + GM_TILE - 1) / GM_TILE);
+    const dim3 grid((rows + GM_TILE - 1) / GM_TILE, g.tiles ? g.max_tiles * ((g.group_columns + GM_TILE - 1) / GM_TILE) : (g.n + GM_TILE - 1) / GM_TILE);
     count_launch();
     return check_cuda(g.w.f32 ? launch_k(dense_gemm_kernel<float>, grid, dim3(256), 0, st, g) : launch_k(dense_gemm_kernel<bf16>, grid, dim3(256), 0, st, g),
                       "dense gemm launch");

@@ -374,7 +374,7 @@ int32_t LayeredModel::build() {
         CERA_CUDA_TRY(cudaMemset(counts, 0, experts * 4));
         CERA_TRY(dev_alloc((void **)&cursor, experts * 4));
         CERA_TRY(dev_alloc((void **)&n_tiles, 8));
-        CERA_TRY(dev_alloc((void **)&tiles, (eo_rows / DENSE_GROUP_COLUMNS + experts) * sizeof(MoeTile)));
+        CERA_TRY(dev_alloc((void **)&tiles, (eo_rows / DENSE_GROUP_MIN + experts) * sizeof(MoeTile)));
         CERA_TRY(dev_alloc(&gathered, eo_rows * gather_w * esz));
         CERA_TRY(dev_alloc(&act, eo_rows * ff_w * esz));
         CERA_TRY(dev_alloc((void **)&eo, eo_rows * ld * 4));
@@ -485,10 +485,10 @@ int32_t LayeredModel::latent_chunk(LayerState &L, size_t n, size_t start_pos) {
 // The routed feed-forward over a chunk: h, h32 -> `eo` in bucket order; `next` sums the picks.
 int32_t LayeredModel::experts_chunk(LayerState &L, size_t n, ResidualNorm *next) {
     const auto &d = L.d;
-    const uint32_t entries = (uint32_t)(n * d.n_used), max_tiles = entries / DENSE_GROUP_COLUMNS + d.n_experts;
+    const uint32_t entries = (uint32_t)(n * d.n_used), columns = dense_group_columns(entries, d.n_experts), max_tiles = entries / columns + d.n_experts;
     CERA_TRY(launch_moe_route(h32, ld, n, (const float *)L.ffn.router.w, nullptr, ld, d.n_experts, d.n_used, d.router_softmax, d.router_renorm, ids, pick_w,
                               counts, stream));
-    CERA_TRY(launch_moe_plan(counts, d.n_experts, DENSE_GROUP_COLUMNS, 0, 0, cursor, tiles, n_tiles, stream));
+    CERA_TRY(launch_moe_plan(counts, d.n_experts, columns, 0, 0, cursor, tiles, n_tiles, stream));
     CERA_TRY(launch_moe_gather(h, f32, ld, ids, pick_w, d.n_used, n, cursor, entry_of, gathered, col_scale, stream));
     DenseGemm g;
     g.w = L.ffn.gate_up;
@@ -501,6 +501,7 @@ int32_t LayeredModel::experts_chunk(LayerState &L, size_t n, ResidualNorm *next)
     g.n_tiles = n_tiles;
     g.max_tiles = max_tiles;
     g.rows_per_expert = 2 * L.ffn.ff_p;
+    g.group_columns = columns;
     g.act = ExpertAct{d.act_limit, d.act_alpha, d.act_shift};
     g.col_scale = d.weight_input ? col_scale : nullptr;
     CERA_TRY(launch_dense_gemm(g, stream));
@@ -514,6 +515,7 @@ int32_t LayeredModel::experts_chunk(LayerState &L, size_t n, ResidualNorm *next)
     o.n_tiles = n_tiles;
     o.max_tiles = max_tiles;
     o.rows_per_expert = ld;
+    o.group_columns = columns;
     CERA_TRY(launch_dense_gemm(o, stream));
     next->y = eo;
     next->entry_of = entry_of;

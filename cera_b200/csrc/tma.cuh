@@ -79,6 +79,14 @@ __device__ __forceinline__ void bulk_g2s(void *dst, const void *src, uint32_t by
                  : "memory");
 }
 
+// A box of a tensor map (the map lives in constant / parameter space) -> this CTA's shared memory; x * element size must be
+// a multiple of 16 bytes.
+__device__ __forceinline__ void tensor_g2s_2d(void *dst, const void *map, int32_t x, int32_t y, uint64_t *bar) {
+    asm volatile("cp.async.bulk.tensor.2d.shared::cluster.global.tile.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4}], [%2];" ::"r"(smem_u32(dst)),
+                 "l"(map), "r"(smem_u32(bar)), "r"(x), "r"(y)
+                 : "memory");
+}
+
 // 16 bytes global -> shared through the LSU's asynchronous copy path (L1-bypassing).
 __device__ __forceinline__ void cp_async16(void *dst, const void *src) {
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
