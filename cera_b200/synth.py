@@ -65,6 +65,57 @@ def build_llama(cfg, seed=0, sigma=0.02, types=None, sink=None, **model_kw):
     return m
 
 
+def goletar_config(width, n_layers, vocab=32768, experts=32, top=4, ff=None):
+    """A Goletar configuration whose layers have the shapes of a real model of this width: minGRU and latent attention in
+    turn, heads of 128 + 64, a latent of 512."""
+    ff = ff or width // 2
+    mlp = {"kind": "moe", "expert": {"ff": ff, "limit": 7.0}, "router": {"experts": experts, "top": top}}
+    gru = {"type": "mingru", "mixer": {"width": width}, "mlp": mlp}
+    att = {"type": "latent_attention", "mlp": mlp,
+           "mixer": {"heads": width // 128, "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": 512, "scale": 192.0 ** -0.5,
+                     "rot": {"base": 10000.0, "dims": 64}}}
+    return {"architecture": "Goletar", "width": width, "vocab": vocab, "norm": {"eps": 1e-6}, "layers": [gru if i % 2 == 0 else att for i in range(n_layers)],
+            "embedding": {"bigram": {"buckets": 100003, "mul_prev": 9973, "mul_cur": 31}}}
+
+
+def build_goletar(config, seed=0, dtype="bfloat16", **model_kw):
+    """A finalized Goletar model with random weights made on the device."""
+    from . import goletar
+    from .layered import Ff, LayeredModel, Mixer
+    from .types import BF16
+    kw, layers = goletar.describe(config)
+    m = LayeredModel(layers, dtype=dtype, **kw, **model_kw)
+    gen = torch.Generator(device="cuda").manual_seed(seed)
+    W = kw["hidden_size"]
+
+    def shape(role, d):
+        if role in (Role.TOKEN_EMBD, Role.OUTPUT):
+            return kw["vocab_size"], W
+        if role == Role.BIGRAM_EMBD:
+            return kw["bigram_buckets"] + 1, W
+        if role in (Role.OUTPUT_NORM, Role.MIX_PRE_NORM, Role.MIX_POST_NORM, Role.FF_PRE_NORM, Role.FF_POST_NORM):
+            return 1, 1
+        latent = d.mixer == Mixer.LATENT_ATTENTION
+        return {Role.MIX_OUTPUT: (W, d.n_heads * d.value_dim if latent else d.recurrent_width),
+                Role.LATENT_Q: (d.n_heads * (d.head_dim + d.rot_dim), W), Role.LATENT_DOWN: (d.kv_rank + d.rot_dim, W), Role.LATENT_NORM: (1, d.kv_rank),
+                Role.LATENT_UP_K: (d.n_heads * d.head_dim, d.kv_rank), Role.LATENT_UP_V: (d.n_heads * d.value_dim, d.kv_rank),
+                Role.LATENT_SINK: (1, d.n_heads), Role.LATENT_GATE: (d.n_heads, W), Role.GRU_Z: (d.recurrent_width, W), Role.GRU_X: (d.recurrent_width, W),
+                Role.GRU_GATE: (d.recurrent_width, W), Role.GRU_Z_BIAS: (1, d.recurrent_width), Role.GRU_X_BIAS: (1, d.recurrent_width),
+                Role.ROUTER: (d.n_experts, W), Role.EXPERT_GATE: (d.ff_width, W), Role.EXPERT_UP: (d.ff_width, W), Role.EXPERT_DOWN: (W, d.ff_width)}[role]
+
+    for _, role, layer, expert in goletar.tensor_roles(layers):
+        rows, cols = shape(role, layers[layer])
+        v = torch.randn(rows, cols, device="cuda", dtype=torch.bfloat16, generator=gen)
+        if rows > 1 and role not in (Role.TOKEN_EMBD, Role.BIGRAM_EMBD):
+            v *= cols ** -0.5
+        elif rows * cols == 1 or role == Role.LATENT_NORM:
+            v.fill_(1.0)
+        m.add_tensor(role, layer, BF16, rows, cols, v, expert=expert)
+    torch.cuda.synchronize()
+    m.finalize()
+    return m
+
+
 def prompt_tokens(n, vocab, seed):
     """Uniform-random token ids, reproducible without numpy's generator state."""
     mask = (1 << 64) - 1

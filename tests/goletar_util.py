@@ -5,7 +5,7 @@ import numpy as np
 
 import goletar_ref as G
 
-F32_TOL, BF16_TOL = 3e-5, 3e-2  # rms over the vocabulary of the logits' difference (mean taken off), in units of their spread
+F32_TOL, BF16_TOL = 1e-5, 2e-2  # rms over the vocabulary of the logits' difference (mean taken off), in units of their spread
 TOL = {"float32": F32_TOL, "bfloat16": BF16_TOL}
 
 
@@ -32,13 +32,14 @@ def tokens(n, vocab, seed):
     return np.random.default_rng(seed).integers(0, vocab, n).tolist()
 
 
-def error(got, want):
-    """Worst position's error."""
+def error(got, want, quantile=1.0):
+    """Worst position's error, or a quantile over the positions: with 16-bit rounding a token whose experts are a close call may
+    go to another one, and a test that routes freely looks at most positions instead of all."""
     got, want = np.asarray(got, dtype=np.float64), np.asarray(want, dtype=np.float64)
     assert got.shape == want.shape and np.isfinite(got).all()
     d = got - want
     d -= d.mean(axis=-1, keepdims=True)
-    return float((np.sqrt((d * d).mean(axis=-1)) / np.maximum(want.std(axis=-1), 1e-6)).max())
+    return float(np.quantile(np.sqrt((d * d).mean(axis=-1)) / np.maximum(want.std(axis=-1), 1e-6), quantile))
 
 
 def aim(cfg, weights, layer, q_tok, k_tok, bump):
