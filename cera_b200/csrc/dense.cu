@@ -45,52 +45,71 @@ __global__ void __launch_bounds__(256) embed_dense_kernel(const T *__restrict__ 
     }
 }
 
-// One CTA per row; the row stays in shared memory between the passes.
-template <class T>
+// One CTA per row, four numbers per thread and vector, the row in registers (V vectors a thread).  The padding of x and y
+// is zero, so whole vectors are summed.
+template <class T, int V>
 __global__ void __launch_bounds__(1024) residual_norm_kernel(ResidualNorm p, uint32_t width, uint32_t ld, float eps) {
-    extern __shared__ float row[];
     __shared__ float red[33];
     pdl_trigger();
     pdl_wait();
-    const uint32_t j = blockIdx.x, t = threadIdx.x, nt = blockDim.x;
-    float *x = p.x + (size_t)(p.x_rows ? p.x_rows[j] : j) * ld;
+    const uint32_t j = blockIdx.x, t = threadIdx.x, nt = blockDim.x, nv = ld / 4;
+    float4 *x = reinterpret_cast<float4 *>(p.x + (size_t)(p.x_rows ? p.x_rows[j] : j) * ld);
     const float inv_w = 1.0f / (float)width;
+    float4 xv[V], yv[V];
     float ss = 0.0f;
-    if (p.y) {
-        for (uint32_t i = t; i < width; i += nt) {
-            float v;
-            if (p.entry_of) {
-                v = 0.0f;
-                for (uint32_t s = 0; s < p.picks; ++s) {
-                    const float e = p.y[(size_t)p.entry_of[j * p.picks + s] * ld + i];
-                    v += p.pick_weight ? e * p.pick_weight[j * p.picks + s] : e;
-                }
-            } else {
-                v = p.y[(size_t)j * ld + i];
-            }
-            row[i] = v;
-            ss += v * v;
-        }
-        const float r = 1.0f / sqrtf(cta_sum(ss, red) * inv_w + eps);
-        ss = 0.0f;
-        for (uint32_t i = t; i < width; i += nt) {
-            const float v = x[i] + row[i] * r * p.post.g[p.post.per_channel ? i : 0];
-            x[i] = v;
-            row[i] = v;
-            ss += v * v;
-        }
-    } else {
-        for (uint32_t i = t; i < width; i += nt) {
-            const float v = x[i];
-            row[i] = v;
-            ss += v * v;
+#pragma unroll
+    for (int e = 0; e < V; ++e) {
+        const uint32_t i = t + e * nt;
+        xv[e] = yv[e] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        if (i < nv) {
+            xv[e] = x[i];
+            if (p.y && !p.entry_of) yv[e] = reinterpret_cast<const float4 *>(p.y + (size_t)j * ld)[i];
         }
     }
+    if (p.y) {
+        if (p.entry_of) {
+            for (uint32_t s = 0; s < p.picks; ++s) {
+                const float4 *row = reinterpret_cast<const float4 *>(p.y + (size_t)p.entry_of[j * p.picks + s] * ld);
+                const float w = p.pick_weight ? p.pick_weight[j * p.picks + s] : 1.0f;
+#pragma unroll
+                for (int e = 0; e < V; ++e)
+                    if (t + e * nt < nv) {
+                        const float4 r = row[t + e * nt];
+                        yv[e].x += w * r.x;
+                        yv[e].y += w * r.y;
+                        yv[e].z += w * r.z;
+                        yv[e].w += w * r.w;
+                    }
+            }
+        }
+#pragma unroll
+        for (int e = 0; e < V; ++e) ss += yv[e].x * yv[e].x + yv[e].y * yv[e].y + yv[e].z * yv[e].z + yv[e].w * yv[e].w;
+        const float r = 1.0f / sqrtf(cta_sum(ss, red) * inv_w + eps);
+#pragma unroll
+        for (int e = 0; e < V; ++e) {
+            const uint32_t i = t + e * nt;
+            if (i < nv) {
+                const float4 g = p.post.at(i);
+                xv[e].x += yv[e].x * r * g.x;
+                xv[e].y += yv[e].y * r * g.y;
+                xv[e].z += yv[e].z * r * g.z;
+                xv[e].w += yv[e].w * r * g.w;
+                x[i] = xv[e];
+            }
+        }
+        ss = 0.0f;
+    }
+#pragma unroll
+    for (int e = 0; e < V; ++e) ss += xv[e].x * xv[e].x + xv[e].y * xv[e].y + xv[e].z * xv[e].z + xv[e].w * xv[e].w;
     const float r = 1.0f / sqrtf(cta_sum(ss, red) * inv_w + eps);
-    for (uint32_t i = t; i < ld; i += nt) {
-        const float v = i < width ? row[i] * r * p.pre.g[p.pre.per_channel ? i : 0] : 0.0f;
-        if (p.h) ((T *)p.h)[(size_t)j * ld + i] = Elem<T>::from(v);
-        if (p.h32) p.h32[(size_t)j * ld + i] = v;
+#pragma unroll
+    for (int e = 0; e < V; ++e) {
+        const uint32_t i = t + e * nt;
+        if (i >= nv) continue;
+        const float4 g = p.pre.at(i);
+        const float4 v = make_float4(xv[e].x * r * g.x, xv[e].y * r * g.y, xv[e].z * r * g.z, xv[e].w * r * g.w);
+        if (p.h) store4((T *)p.h + (size_t)j * ld + 4 * i, v);
+        if (p.h32) reinterpret_cast<float4 *>(p.h32 + (size_t)j * ld)[i] = v;
     }
 }
 
@@ -139,16 +158,28 @@ int32_t launch_embed_dense(const DenseView &table, const DenseView &bigram, cons
 
 int32_t launch_residual_norm(const ResidualNorm &p, uint32_t width, uint32_t ld, size_t n, float eps, cudaStream_t st) {
     if (n == 0) return CERA_CUDA_OK;
-    const size_t smem = (size_t)width * 4;
-    if (smem > 200 * 1024) return fail(CERA_CUDA_ERR_UNSUPPORTED, "norm: rows of %u numbers", width);
-    uint32_t threads = n == 1 ? 1024u : 256u;
-    while (threads > 64 && threads / 2 >= width) threads /= 2;
-    auto go = [&](auto kernel) -> int32_t {
-        if (smem > 48 * 1024) CERA_CUDA_TRY(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+    const uint32_t nv = ld / 4;
+    // one vector a thread for a lone row, four for many
+    uint32_t v = n == 1 ? 1 : 4;
+    while (v > 1 && nv < v * 32) v /= 2;
+    while (v < 16 && (nv + v - 1) / v > 1024) v *= 2;
+    const uint32_t threads = ((nv + v - 1) / v + 31) / 32 * 32;
+    if (threads > 1024) return fail(CERA_CUDA_ERR_UNSUPPORTED, "norm: rows of %u numbers (at most 65536)", width);
+    auto go = [&](auto kernel) {
         count_launch();
-        return check_cuda(launch_k(kernel, dim3((unsigned)n), dim3(threads), smem, st, p, width, ld, eps), "residual norm launch");
+        return check_cuda(launch_k(kernel, dim3((unsigned)n), dim3(threads), 0, st, p, width, ld, eps), "residual norm launch");
     };
-    return p.h_f32 ? go(residual_norm_kernel<float>) : go(residual_norm_kernel<bf16>);
+    auto typed = [&](auto t) {
+        using T = decltype(t);
+        switch (v) {
+            case 1: return go(residual_norm_kernel<T, 1>);
+            case 2: return go(residual_norm_kernel<T, 2>);
+            case 4: return go(residual_norm_kernel<T, 4>);
+            case 8: return go(residual_norm_kernel<T, 8>);
+            default: return go(residual_norm_kernel<T, 16>);
+        }
+    };
+    return p.h_f32 ? typed(float{}) : typed(bf16{});
 }
 
 int32_t launch_moe_gather(const void *h, int f32, uint32_t ld, const uint32_t *ids, const float *weights, uint32_t n_used, size_t n, uint32_t *cursor,

@@ -36,8 +36,14 @@ struct Elem<float> {
     static __device__ __forceinline__ float from(float v) { return v; }
 };
 
-__device__ __forceinline__ float sigmoid_f32(float x) { return 1.0f / (1.0f + expf(-x)); }
-__device__ __forceinline__ float silu_f32(float x) { return x / (1.0f + expf(-x)); }
+__device__ __forceinline__ void store4(float *p, const float4 &v) { *reinterpret_cast<float4 *>(p) = v; }
+__device__ __forceinline__ void store4(bf16 *p, const float4 &v) {
+    const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+    *reinterpret_cast<uint2 *>(p) = make_uint2(*reinterpret_cast<const uint32_t *>(&a), *reinterpret_cast<const uint32_t *>(&b));
+}
+
+__device__ __forceinline__ float sigmoid_f32(float x) { return __fdividef(1.0f, 1.0f + expf(-x)); }
+__device__ __forceinline__ float silu_f32(float x) { return x * sigmoid_f32(x); }
 // min(g, limit) * sigmoid(alpha g) * (clamp(u) + shift)
 __device__ __forceinline__ float gated_unit(float g, float u, const ExpertAct &a) {
     g = fminf(g, a.limit);

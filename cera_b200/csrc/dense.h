@@ -19,10 +19,15 @@ struct DenseView {
 
 inline uint32_t pad_to(uint32_t v, uint32_t a) { return (v + a - 1) / a * a; }
 
-// A norm: g holds one number (per_channel 0) or one per channel (1).
+// A norm: g holds one number (per_channel 0) or one per channel (1, the row length's padding included).
 struct NormView {
     const float *g = nullptr;
     int per_channel = 0;
+    __device__ __forceinline__ float4 at(uint32_t i4) const {  // of channels 4 i4 .. 4 i4 + 3
+        if (per_channel) return reinterpret_cast<const float4 *>(g)[i4];
+        const float v = *g;
+        return make_float4(v, v, v, v);
+    }
 };
 
 // Index i of a padded axis: groups of `group` source entries become groups of `group_p`, of which the first `seg`

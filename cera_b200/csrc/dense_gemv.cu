@@ -165,26 +165,44 @@ __global__ void __launch_bounds__(GV_WARPS * 32) expert_down_kernel(const T *__r
     pdl_wait();
     const int warp = threadIdx.x >> 5;
     const uint32_t g = blockIdx.x * (GV_WARPS / WPR) + warp / WPR, gi = min(g, rows - 1);
+    // the picks' rows are walked as one row of n_used * ld elements, U vectors of it in flight per lane
+    constexpr int U = 8;
+    const uint32_t nv = ld / Elem<T>::N, all = n_used * nv, step = 32u * WPR;
     float total[1] = {0.0f};
-    for (uint32_t s = 0; s < n_used; ++s) {
-        RowDot<T, 1, 8> d;
-        d.w[0] = w + ((size_t)ids[s] * rows + gi) * ld;
-        d.start(ld, warp % WPR, WPR);
-        d.fetch();
-        float acc[1] = {0.0f};
-        d.run(act + (size_t)s * ld, acc);
-        total[0] += weight_input ? acc[0] : weights[s] * acc[0];
+    for (uint32_t c = (warp % WPR) * 32u + (threadIdx.x & 31); c < all; c += U * step) {
+        uint4 wb[U], xb[U];
+        float sc[U];
+#pragma unroll
+        for (int u = 0; u < U; ++u) {
+            const uint32_t v = c + u * step, s = v / nv;
+            if (v < all) {
+                wb[u] = ld_stream(reinterpret_cast<const uint4 *>(w + ((size_t)ids[s] * rows + gi) * ld) + (v - s * nv));
+                xb[u] = *(reinterpret_cast<const uint4 *>(act) + v);
+                sc[u] = weight_input ? 1.0f : weights[s];
+            }
+        }
+#pragma unroll
+        for (int u = 0; u < U; ++u)
+            if (c + u * step < all) {
+                float wf[Elem<T>::N], xf[Elem<T>::N], a = 0.0f;
+                Elem<T>::unpack(wb[u], wf);
+                Elem<T>::unpack(xb[u], xf);
+#pragma unroll
+                for (int i = 0; i < Elem<T>::N; ++i) a = fmaf(wf[i], xf[i], a);
+                total[0] = fmaf(sc[u], a, total[0]);
+            }
     }
     group_sum<1, WPR>(total, red);
     if (warp % WPR == 0 && (threadIdx.x & 31) == 0 && g < rows) y[g] = total[0];
 }
 
-// Warps per row group: enough warps to cover the memory latency when there are few groups.
-int pick_wpr(size_t groups) {
-    const size_t want = (size_t)sm_count() * 14;
-    for (int wpr = 1; wpr < 8; wpr *= 2)
-        if (groups * wpr >= want) return wpr;
-    return 8;
+// Warps per row group: shared further while every warp keeps a batch of loads (u vectors a lane) and all groups still run
+// at once; few groups are shared whatever the batch.
+int pick_wpr(size_t groups, size_t row_bytes, int u) {
+    const size_t vecs = row_bytes / 16, few = (size_t)sm_count() * 14, room = (size_t)sm_count() * 64;
+    int wpr = 1;
+    while (wpr < 8 && (groups * wpr < few || (groups * wpr * 2 <= room && vecs >= (size_t)wpr * 2 * 32 * u))) wpr *= 2;
+    return wpr;
 }
 
 template <class F>
@@ -207,7 +225,7 @@ dim3 gv_grid(size_t groups, int wpr, uint32_t y = 1) { return dim3((unsigned)((g
 int32_t launch_dense_gemv(const DenseView &w, const void *x, float *y, cudaStream_t st) {
     const bool two = w.rows >= (uint32_t)sm_count() * 28;
     const size_t groups = two ? (w.rows + 1) / 2 : w.rows;
-    const int wpr = pick_wpr(groups);
+    const int wpr = pick_wpr(groups, (size_t)w.ld * (w.f32 ? 4 : 2), two ? 4 : 8);
     count_launch();
     return with_type(w.f32, [&](auto t) {
         using T = decltype(t);
@@ -222,7 +240,7 @@ int32_t launch_dense_gemv(const DenseView &w, const void *x, float *y, cudaStrea
 
 int32_t launch_mingru_step(const DenseView &w, const void *x, const float *z_bias, const float *x_bias, float *state, void *out, cudaStream_t st) {
     const uint32_t wp = w.rows / 3;
-    const int wpr = pick_wpr(wp);
+    const int wpr = pick_wpr(wp, (size_t)w.ld * (w.f32 ? 4 : 2), 4);
     count_launch();
     return with_type(w.f32, [&](auto t) {
         using T = decltype(t);
@@ -236,7 +254,7 @@ int32_t launch_mingru_step(const DenseView &w, const void *x, const float *z_bia
 
 int32_t launch_expert_gate_up_step(const DenseView &w, const void *x, const float *router_logits, const RouterRule &r, uint32_t ff_p, const ExpertAct &a,
                                    uint32_t *ids, float *weights, void *act, cudaStream_t st) {
-    const int wpr = pick_wpr((size_t)ff_p * r.n_used);
+    const int wpr = pick_wpr((size_t)ff_p * r.n_used, (size_t)w.ld * (w.f32 ? 4 : 2), 4);
     count_launch();
     return with_type(w.f32, [&](auto t) {
         using T = decltype(t);
@@ -250,7 +268,7 @@ int32_t launch_expert_gate_up_step(const DenseView &w, const void *x, const floa
 
 int32_t launch_expert_down_step(const DenseView &w, uint32_t rows_per_expert, const void *act, const RouterRule &r, const uint32_t *ids,
                                 const float *weights, float *y, cudaStream_t st) {
-    const int wpr = pick_wpr(rows_per_expert);
+    const int wpr = pick_wpr(rows_per_expert, (size_t)w.ld * (w.f32 ? 4 : 2), 2);
     count_launch();
     return with_type(w.f32, [&](auto t) {
         using T = decltype(t);

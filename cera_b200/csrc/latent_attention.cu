@@ -9,7 +9,7 @@ namespace cera {
 
 namespace {
 
-// One CTA per token.
+// grid (tokens, parts): part 0 takes the latent, the rotated key part and the gates, the others a share of q.
 template <class T>
 __global__ void __launch_bounds__(256) latent_prepare_kernel(const float *in, LatentShape s, uint32_t start_pos, const uint32_t *pos_dev,
                                                              const float *__restrict__ c_norm, float eps, const float *__restrict__ rope, T *cache_c,
@@ -20,24 +20,28 @@ __global__ void __launch_bounds__(256) latent_prepare_kernel(const float *in, La
     const uint32_t j = blockIdx.x, pos = (pos_dev ? *pos_dev : start_pos) + j, t = threadIdx.x;
     const float *row = in + (size_t)j * s.in_p, *c = row + s.off_c(), *kr = row + s.off_r(), *gl = row + s.off_g();
     const float *cs = rope + (size_t)pos * s.rot;  // (cos, sin) of the rot / 2 pairs
-    float ss = 0.0f;
-    for (uint32_t i = t; i < s.rank; i += 256) ss += c[i] * c[i];
-    const float r = 1.0f / sqrtf(cta_sum(ss, red) / (float)s.rank + eps);
-    for (uint32_t i = t; i < s.rank_p; i += 256) cache_c[(size_t)pos * s.rank_p + i] = Elem<T>::from(c[i] * r * c_norm[i]);
     auto turned = [&](const float *v, uint32_t i) {  // element i of the rotated vector
         if (i >= s.rot) return 0.0f;
         const float cv = cs[i & ~1u], sv = cs[i | 1u];
         return i & 1 ? v[i] * cv + v[i - 1] * sv : v[i] * cv - v[i + 1] * sv;
     };
-    for (uint32_t i = t; i < s.rot_p; i += 256) cache_r[(size_t)pos * s.rot_p + i] = Elem<T>::from(turned(kr, i));
+    if (blockIdx.y == 0) {
+        float ss = 0.0f;
+        for (uint32_t i = t; i < s.rank; i += 256) ss += c[i] * c[i];
+        const float r = 1.0f / sqrtf(cta_sum(ss, red) / (float)s.rank + eps);
+        for (uint32_t i = t; i < s.rank_p; i += 256) cache_c[(size_t)pos * s.rank_p + i] = Elem<T>::from(c[i] * r * c_norm[i]);
+        for (uint32_t i = t; i < s.rot_p; i += 256) cache_r[(size_t)pos * s.rot_p + i] = Elem<T>::from(turned(kr, i));
+        for (uint32_t h = t; h < s.heads; h += 256) gate[(size_t)j * s.heads + h] = sigmoid_f32(gl[h]);
+        return;
+    }
     const uint32_t hd = s.dim_p + s.rot_p, total = s.heads * hd;
-    for (uint32_t i = t; i < total; i += 256) {
+#pragma unroll 4
+    for (uint32_t i = (blockIdx.y - 1) * 256 + t; i < total; i += (gridDim.y - 1) * 256) {
         const uint32_t d = i % hd;
         const float v = d < s.dim_p ? row[i] : turned(row + (i - d) + s.dim_p, d - s.dim_p);
         if (q32) q32[(size_t)j * total + i] = v;
         if (qt) qt[(size_t)j * total + i] = Elem<T>::from(v);
     }
-    for (uint32_t h = t; h < s.heads; h += 256) gate[(size_t)j * s.heads + h] = sigmoid_f32(gl[h]);
 }
 
 // q_lat[j][h] = [W_uk_h^T q_h, rotated part].  grid (64-column slabs of rank_p, heads, queries), 4 x 64 threads: thread
@@ -45,15 +49,22 @@ __global__ void __launch_bounds__(256) latent_prepare_kernel(const float *in, La
 template <class T>
 __global__ void __launch_bounds__(256) latent_query_kernel(const float *q32, LatentShape s, const T *__restrict__ uk, float *q_lat) {
     __shared__ float part[4][64];
+    constexpr int PRE = 32;  // weights fetched ahead of the wait
     pdl_trigger();
-    pdl_wait();
     const uint32_t h = blockIdx.y, j = blockIdx.z, col = threadIdx.x & 63, sl = threadIdx.x >> 6, c = blockIdx.x * 64 + col;
     const uint32_t hd = s.dim_p + s.rot_p, ldo = s.rank_p + s.rot_p;
     const float *q = q32 + ((size_t)j * s.heads + h) * hd;
     const T *w = uk + (size_t)h * s.dim_p * s.rank_p + c;
+    T ahead[PRE];
+#pragma unroll
+    for (int i = 0; i < PRE; ++i)
+        if (sl + 4 * i < s.dim_p) ahead[i] = w[(size_t)(sl + 4 * i) * s.rank_p];
+    pdl_wait();
     float acc = 0.0f;
-#pragma unroll 8
-    for (uint32_t d = sl; d < s.dim_p; d += 4) acc = fmaf(q[d], Elem<T>::to(w[(size_t)d * s.rank_p]), acc);
+#pragma unroll
+    for (int i = 0; i < PRE; ++i)
+        if (sl + 4 * i < s.dim_p) acc = fmaf(q[sl + 4 * i], Elem<T>::to(ahead[i]), acc);
+    for (uint32_t d = sl + 4 * PRE; d < s.dim_p; d += 4) acc = fmaf(q[d], Elem<T>::to(w[(size_t)d * s.rank_p]), acc);
     part[sl][col] = acc;
     __syncthreads();
     float *o = q_lat + ((size_t)j * s.heads + h) * ldo;
@@ -79,19 +90,22 @@ __global__ void __launch_bounds__(LA_WARPS * 32) latent_split_kernel(const float
     const uint32_t split = blockIdx.x, h0 = blockIdx.y * LA_WARPS * HG, j = blockIdx.z, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const uint32_t len = len_dev ? *len_dev : start_pos + j + 1;
     const uint32_t per = ((len + splits - 1) / splits + LA_KEYS - 1) / LA_KEYS * LA_KEYS, k0 = min(split * per, len), k1 = min(k0 + per, len);
-    for (uint32_t i = threadIdx.x; i < LA_WARPS * HG * ql; i += LA_WARPS * 32) {
-        const uint32_t h = h0 + i / ql;
-        qs[i] = h < s.heads ? q_lat[((size_t)j * s.heads + h) * ql + i % ql] : 0.0f;
+    {
+        const uint32_t live = min((uint32_t)(LA_WARPS * HG), s.heads - h0) * ql / 4;  // the heads of this CTA are one range
+        const float4 *src = reinterpret_cast<const float4 *>(q_lat + ((size_t)j * s.heads + h0) * ql);
+        for (uint32_t i = threadIdx.x; i < LA_WARPS * HG * ql / 4; i += LA_WARPS * 32) {
+            if (i < live) tma::cp_async16(qs + 4 * i, src + i);
+            else *reinterpret_cast<float4 *>(qs + 4 * i) = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        }
     }
-    auto fetch = [&](uint32_t base, int stage) {
+    auto fetch = [&](uint32_t base, int stage) {  // warp = key, lane = vector
         uint8_t *dst = tile + (size_t)stage * LA_KEYS * row_b;
-        for (uint32_t i = threadIdx.x; i < LA_KEYS * row_v; i += LA_WARPS * 32) {
-            const uint32_t k = i / row_v, v = i - k * row_v;
-            if (base + k < k1) {
-                const T *src = v < c_v ? cache_c + (size_t)(base + k) * s.rank_p + v * VN : cache_r + (size_t)(base + k) * s.rot_p + (v - c_v) * VN;
-                tma::cp_async16(dst + (size_t)k * row_b + v * 16, src);
-            } else {
-                *reinterpret_cast<uint4 *>(dst + (size_t)k * row_b + v * 16) = make_uint4(0, 0, 0, 0);
+#pragma unroll 4
+        for (uint32_t k = warp; k < LA_KEYS; k += LA_WARPS) {
+            const T *cr = cache_c + (size_t)(base + k) * s.rank_p, *rr = cache_r + (size_t)(base + k) * s.rot_p;
+            for (uint32_t v = lane; v < row_v; v += 32) {
+                if (base + k < k1) tma::cp_async16(dst + (size_t)k * row_b + v * 16, v < c_v ? cr + v * VN : rr + (v - c_v) * VN);
+                else *reinterpret_cast<uint4 *>(dst + (size_t)k * row_b + v * 16) = make_uint4(0, 0, 0, 0);
             }
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
@@ -213,6 +227,7 @@ __global__ void __launch_bounds__(256) latent_merge_kernel(const float *part, La
     __syncthreads();
     for (uint32_t c = threadIdx.x; c < s.rank_p; c += 256) {
         float v = 0.0f;
+#pragma unroll 8
         for (uint32_t i = 0; i < splits; ++i) v = fmaf(wt[i], p[(size_t)i * ps + 2 + c], v);
         lat[c] = v;
     }
@@ -285,11 +300,13 @@ uint32_t latent_splits(size_t n_positions) {
 int32_t launch_latent_prepare(const float *in, const LatentShape &s, size_t n, size_t start_pos, const uint32_t *pos_dev, const float *c_norm, float eps,
                               const float *rope_table, void *cache_c, void *cache_r, int f32, float *q32, void *qt, float *gate, cudaStream_t st) {
     if (n == 0) return CERA_CUDA_OK;
+    const uint32_t total = s.q_ld(), per = n == 1 ? 512 : 2048;  // q elements of a CTA
+    const dim3 grid((unsigned)n, 1 + (total + per - 1) / per);
     count_launch();
     if (f32)
-        return check_cuda(launch_k(latent_prepare_kernel<float>, dim3((unsigned)n), dim3(256), 0, st, in, s, (uint32_t)start_pos, pos_dev, c_norm, eps,
+        return check_cuda(launch_k(latent_prepare_kernel<float>, grid, dim3(256), 0, st, in, s, (uint32_t)start_pos, pos_dev, c_norm, eps,
                                    rope_table, (float *)cache_c, (float *)cache_r, q32, (float *)qt, gate), "latent prepare launch");
-    return check_cuda(launch_k(latent_prepare_kernel<bf16>, dim3((unsigned)n), dim3(256), 0, st, in, s, (uint32_t)start_pos, pos_dev, c_norm, eps, rope_table,
+    return check_cuda(launch_k(latent_prepare_kernel<bf16>, grid, dim3(256), 0, st, in, s, (uint32_t)start_pos, pos_dev, c_norm, eps, rope_table,
                                (bf16 *)cache_c, (bf16 *)cache_r, q32, (bf16 *)qt, gate), "latent prepare launch");
 }
 

@@ -216,7 +216,7 @@ int32_t LayeredModel::add_tensor(int32_t role, int32_t layer, int32_t type, size
         const size_t n = rows * cols;
         if (n != 1 && n != W) return fail(CERA_CUDA_ERR_BAD_ARG, "add_tensor: norm of role %d layer %d has %zu numbers", role, layer, n);
         float *p = nullptr;
-        CERA_TRY(vec(&p, (uint32_t)n));
+        CERA_TRY(vec(&p, n > 1 ? ld : 1));
         nv->g = p;
         nv->per_channel = n > 1 || W == 1;
         return vector(p, n);

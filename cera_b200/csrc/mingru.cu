@@ -8,7 +8,7 @@ namespace cera {
 
 namespace {
 
-constexpr int SCAN_WARPS = 32;
+constexpr int SCAN_WARPS = 32, SCAN_U = 8;
 
 template <class T>
 __global__ void __launch_bounds__(SCAN_WARPS * 32) mingru_scan_kernel(const float *pre, uint32_t n, uint32_t wp, const float *__restrict__ zb,
@@ -20,25 +20,49 @@ __global__ void __launch_bounds__(SCAN_WARPS * 32) mingru_scan_kernel(const floa
     const uint32_t seg = (n + SCAN_WARPS - 1) / SCAN_WARPS, t0 = min(warp * seg, n), t1 = min(t0 + seg, n);
     const float bz = zb[c], bx = xb[c];
     const size_t ld = 3 * (size_t)wp;
+    // raw products of U tokens at a time: the loads go out together
+    auto walk = [&](auto step) {
+        for (uint32_t t = t0; t < t1; t += SCAN_U) {
+            float zr[SCAN_U], ur[SCAN_U];
+#pragma unroll
+            for (int u = 0; u < SCAN_U; ++u) {
+                const bool in = t + u < t1;
+                zr[u] = in ? pre[(t + u) * ld + c] : 0.0f;
+                ur[u] = in ? pre[(t + u) * ld + wp + c] : 0.0f;
+            }
+            step(t, zr, ur);
+        }
+    };
     float A = 1.0f, B = 0.0f;
-    for (uint32_t t = t0; t < t1; ++t) {
-        float z, cand;
-        mingru_gates(pre[t * ld + c], pre[t * ld + wp + c], bz, bx, z, cand);
-        A *= 1.0f - z;
-        B = (1.0f - z) * B + z * cand;
-    }
+    walk([&](uint32_t t, const float *zr, const float *ur) {
+#pragma unroll
+        for (int u = 0; u < SCAN_U; ++u)
+            if (t + u < t1) {
+                float z, cand;
+                mingru_gates(zr[u], ur[u], bz, bx, z, cand);
+                A *= 1.0f - z;
+                B = (1.0f - z) * B + z * cand;
+            }
+    });
     sa[warp][lane] = A;
     sb[warp][lane] = B;
     const float s0 = state[c];
     __syncthreads();
     float s = s0;
     for (uint32_t w = 0; w < warp; ++w) s = sa[w][lane] * s + sb[w][lane];
-    for (uint32_t t = t0; t < t1; ++t) {
-        float z, cand;
-        mingru_gates(pre[t * ld + c], pre[t * ld + wp + c], bz, bx, z, cand);
-        s = (1.0f - z) * s + z * cand;
-        out[(size_t)t * wp + c] = Elem<T>::from(s * silu_f32(pre[t * ld + 2 * wp + c]));
-    }
+    walk([&](uint32_t t, const float *zr, const float *ur) {
+        float gr[SCAN_U];
+#pragma unroll
+        for (int u = 0; u < SCAN_U; ++u) gr[u] = t + u < t1 ? pre[(t + u) * ld + 2 * wp + c] : 0.0f;
+#pragma unroll
+        for (int u = 0; u < SCAN_U; ++u)
+            if (t + u < t1) {
+                float z, cand;
+                mingru_gates(zr[u], ur[u], bz, bx, z, cand);
+                s = (1.0f - z) * s + z * cand;
+                out[(size_t)(t + u) * wp + c] = Elem<T>::from(s * silu_f32(gr[u]));
+            }
+    });
     if (t1 == n && t0 < n) state[c] = s;  // the warp that holds the last token
 }
 

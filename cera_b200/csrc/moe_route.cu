@@ -6,34 +6,47 @@ namespace cera {
 
 namespace {
 
-// One CTA per token.  Warps take experts round-robin; lane-strided f32 dot, shuffle tree.
+// One CTA per T tokens.  Warps take experts round-robin; lane-strided f32 dots (a router element is loaded once for the T
+// tokens), shuffle tree; then warp t picks for token t.
+template <int T>
 __global__ void __launch_bounds__(256) moe_route_kernel(const float *x, const float *__restrict__ router,
-                                                        const float *__restrict__ bias, uint32_t hidden, uint32_t ld_x, uint32_t n_expert,
+                                                        const float *__restrict__ bias, uint32_t hidden, uint32_t ld_x, uint32_t n, uint32_t n_expert,
                                                         uint32_t n_used, int softmax_gate, int renorm, uint32_t *ids, float *weights,
                                                         uint32_t *counts) {
-    __shared__ float probs[MOE_MAX_EXPERTS];
-    __shared__ uint32_t picked[MOE_MAX_USED];
-    __shared__ float w[MOE_MAX_USED];
+    __shared__ float probs[T][MOE_MAX_EXPERTS];
+    __shared__ uint32_t picked[T][MOE_MAX_USED];
+    __shared__ float w[T][MOE_MAX_USED];
     pdl_trigger();
     pdl_wait();
-    const uint32_t j = blockIdx.x;
+    const uint32_t j0 = blockIdx.x * T;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    const float *xj = x + (size_t)j * ld_x;
+    const float *xj[T];
+#pragma unroll
+    for (int t = 0; t < T; ++t) xj[t] = x + (size_t)min(j0 + t, n - 1) * ld_x;
     for (uint32_t e = warp; e < n_expert; e += blockDim.x >> 5) {
         const float *r = router + (size_t)e * hidden;
-        float acc = 0.0f;
-        for (uint32_t i = lane; i < hidden; i += 32) acc = fmaf(r[i], xj[i], acc);
-        acc = warp_sum(acc);
-        if (lane == 0) probs[e] = acc;
+        float acc[T] = {};
+        for (uint32_t i = lane; i < hidden; i += 32) {
+            const float rv = r[i];
+#pragma unroll
+            for (int t = 0; t < T; ++t) acc[t] = fmaf(rv, xj[t][i], acc[t]);
+        }
+#pragma unroll
+        for (int t = 0; t < T; ++t) {
+            acc[t] = warp_sum(acc[t]);
+            if (lane == 0) probs[t][e] = acc[t];
+        }
     }
     __syncthreads();
-    moe_scores(probs, n_expert, softmax_gate);
-    if (warp != 0) return;
-    moe_pick(probs, bias, n_expert, n_used, renorm, picked, w);
+#pragma unroll 1
+    for (int t = 0; t < T; ++t) moe_scores(probs[t], n_expert, softmax_gate);
+    if (warp >= T || j0 + warp >= n) return;
+    const uint32_t j = j0 + warp;
+    moe_pick(probs[warp], bias, n_expert, n_used, renorm, picked[warp], w[warp]);
     if (lane < n_used) {
-        ids[(size_t)j * n_used + lane] = picked[lane];
-        weights[(size_t)j * n_used + lane] = w[lane];
-        atomicAdd(counts + picked[lane], 1u);
+        ids[(size_t)j * n_used + lane] = picked[warp][lane];
+        weights[(size_t)j * n_used + lane] = w[warp][lane];
+        atomicAdd(counts + picked[warp][lane], 1u);
     }
 }
 
@@ -43,14 +56,19 @@ __global__ void moe_plan_kernel(uint32_t *counts, uint32_t n_expert, uint32_t nc
                                 MoeTile *tiles, uint32_t *n_tiles) {
     pdl_trigger();
     pdl_wait();
+    __shared__ uint32_t n_of[MOE_MAX_EXPERTS];
+    for (uint32_t e = threadIdx.x; e < n_expert; e += blockDim.x) {
+        n_of[e] = counts[e];
+        counts[e] = 0;
+    }
+    __syncthreads();
     if (threadIdx.x != 0) return;
     uint32_t off = 0, t = 0, ts = 0;
     for (uint32_t e = 0; e < n_expert; ++e) {
-        const uint32_t c = counts[e];
+        const uint32_t c = n_of[e];
         cursor[e] = off;
         moe_emit_items(tiles, cap, t, ts, e, off, c, nc, small_nc);
         off += c;
-        counts[e] = 0;
     }
     n_tiles[0] = t;
     n_tiles[1] = ts;
@@ -64,9 +82,12 @@ int32_t launch_moe_route(const float *x, size_t ld_x, size_t n, const float *rou
         return fail(CERA_CUDA_ERR_BAD_ARG, "moe route: %u experts, %u used (limits %d, %d)", n_expert, n_used, MOE_MAX_EXPERTS, MOE_MAX_USED);
     if (n == 0) return CERA_CUDA_OK;
     count_launch();
-    return check_cuda(launch_k(moe_route_kernel, dim3((unsigned)n), dim3(256), 0, st, x, router, bias, hidden, (uint32_t)ld_x, n_expert, n_used,
-                               softmax_gate, renorm, ids, weights, counts),
-                      "moe route launch");
+    auto go = [&](auto kernel, uint32_t per) {
+        return check_cuda(launch_k(kernel, dim3((unsigned)((n + per - 1) / per)), dim3(256), 0, st, x, router, bias, hidden, (uint32_t)ld_x, (uint32_t)n, n_expert,
+                                   n_used, softmax_gate, renorm, ids, weights, counts),
+                          "moe route launch");
+    };
+    return n < (size_t)sm_count() * 4 ? go(moe_route_kernel<1>, 1) : go(moe_route_kernel<8>, 8);
 }
 
 int32_t launch_moe_plan(uint32_t *counts, uint32_t n_expert, uint32_t nc, uint32_t small_nc, uint32_t cap, uint32_t *cursor, MoeTile *tiles,
