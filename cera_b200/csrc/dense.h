@@ -148,7 +148,7 @@ struct LatentScratch {
     float *q_lat = nullptr;  // [queries][heads][rank_p + rot_p]
     float *part = nullptr;   // [queries][heads][splits][rank_p + 2]
 };
-constexpr uint32_t LATENT_MAX_SPLITS = 64;  // queries * splits of one call never exceed this
+constexpr uint32_t LATENT_MAX_SPLITS = 128;  // queries * splits of one call never exceed this
 uint32_t latent_splits(size_t n_positions);
 int32_t launch_latent_attention(const float *q32, const LatentShape &s, const DenseView &uk, const DenseView &uv, const void *cache_c, const void *cache_r,
                                 const float *sink, const float *gate, size_t n, size_t start_pos, const uint32_t *len_dev, uint32_t splits,

@@ -2,8 +2,14 @@
 // rotated key part per position are cached.  This file: what every path needs (norm, rotation, cache append) and the
 // latent-space form, in which W_uk is applied to the query and W_uv to the weighted sum of latents - the decode step,
 // short prompt portions, and everything in f32.  Scores, softmax and sums are f32.
+#include <cooperative_groups.h>
+
+#include <type_traits>
+
 #include "dense.cuh"
 #include "tma.cuh"
+
+namespace cg = cooperative_groups;
 
 namespace cera {
 
@@ -44,33 +50,49 @@ __global__ void __launch_bounds__(256) latent_prepare_kernel(const float *in, La
     }
 }
 
-// q_lat[j][h] = [W_uk_h^T q_h, rotated part].  grid (64-column slabs of rank_p, heads, queries), 4 x 64 threads: thread
-// (slice of the head's dimensions, column).
+// q_lat[j][h] = [W_uk_h^T q_h, rotated part].  grid (64-column slabs of rank_p, heads, queries), 256 threads = 16 slices of
+// the head's dimensions x 16 groups of four columns; weights are fetched ahead of the wait.
 template <class T>
 __global__ void __launch_bounds__(256) latent_query_kernel(const float *q32, LatentShape s, const T *__restrict__ uk, float *q_lat) {
-    __shared__ float part[4][64];
-    constexpr int PRE = 32;  // weights fetched ahead of the wait
+    using V = typename std::conditional<sizeof(T) == 2, uint2, uint4>::type;  // four elements
+    __shared__ float4 part[16][16];
+    constexpr int PRE = 8;
     pdl_trigger();
-    const uint32_t h = blockIdx.y, j = blockIdx.z, col = threadIdx.x & 63, sl = threadIdx.x >> 6, c = blockIdx.x * 64 + col;
+    const uint32_t h = blockIdx.y, j = blockIdx.z, cg = threadIdx.x & 15, sl = threadIdx.x >> 4, c = blockIdx.x * 64 + cg * 4;
     const uint32_t hd = s.dim_p + s.rot_p, ldo = s.rank_p + s.rot_p;
     const float *q = q32 + ((size_t)j * s.heads + h) * hd;
     const T *w = uk + (size_t)h * s.dim_p * s.rank_p + c;
-    T ahead[PRE];
+    V ahead[PRE];
 #pragma unroll
     for (int i = 0; i < PRE; ++i)
-        if (sl + 4 * i < s.dim_p) ahead[i] = w[(size_t)(sl + 4 * i) * s.rank_p];
+        if (sl + 16 * i < s.dim_p) ahead[i] = *reinterpret_cast<const V *>(w + (size_t)(sl + 16 * i) * s.rank_p);
     pdl_wait();
-    float acc = 0.0f;
+    float4 acc = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    auto add = [&](const V &v, float qv) {
+        const T *e = reinterpret_cast<const T *>(&v);
+        acc.x = fmaf(qv, Elem<T>::to(e[0]), acc.x);
+        acc.y = fmaf(qv, Elem<T>::to(e[1]), acc.y);
+        acc.z = fmaf(qv, Elem<T>::to(e[2]), acc.z);
+        acc.w = fmaf(qv, Elem<T>::to(e[3]), acc.w);
+    };
+    float qv[PRE];
+#pragma unroll
+    for (int i = 0; i < PRE; ++i) qv[i] = sl + 16 * i < s.dim_p ? q[sl + 16 * i] : 0.0f;
 #pragma unroll
     for (int i = 0; i < PRE; ++i)
-        if (sl + 4 * i < s.dim_p) acc = fmaf(q[sl + 4 * i], Elem<T>::to(ahead[i]), acc);
-    for (uint32_t d = sl + 4 * PRE; d < s.dim_p; d += 4) acc = fmaf(q[d], Elem<T>::to(w[(size_t)d * s.rank_p]), acc);
-    part[sl][col] = acc;
+        if (sl + 16 * i < s.dim_p) add(ahead[i], qv[i]);
+    for (uint32_t d = sl + 16 * PRE; d < s.dim_p; d += 16) add(*reinterpret_cast<const V *>(w + (size_t)d * s.rank_p), q[d]);
+    part[sl][cg] = acc;
     __syncthreads();
     float *o = q_lat + ((size_t)j * s.heads + h) * ldo;
-    if (sl == 0) o[c] = part[0][col] + part[1][col] + part[2][col] + part[3][col];
-    if (blockIdx.x == 0)
-        for (uint32_t i = threadIdx.x; i < s.rot_p; i += 256) o[s.rank_p + i] = q[s.dim_p + i];
+    if (threadIdx.x < 64) {
+        float v = 0.0f;
+#pragma unroll
+        for (int i = 0; i < 16; ++i) v += reinterpret_cast<const float *>(part[i])[threadIdx.x];
+        o[blockIdx.x * 64 + threadIdx.x] = v;
+    } else if (blockIdx.x == 0) {
+        for (uint32_t i = threadIdx.x - 64; i < s.rot_p; i += 192) o[s.rank_p + i] = q[s.dim_p + i];
+    }
 }
 
 constexpr int LA_WARPS = 4, LA_KEYS = 32;
@@ -132,6 +154,7 @@ __global__ void __launch_bounds__(LA_WARPS * 32) latent_split_kernel(const float
 #pragma unroll
         for (int g = 0; g < HG; ++g) sc[g] = 0.0f;
         const uint4 *kv = reinterpret_cast<const uint4 *>(tl + (size_t)lane * row_b);
+#pragma unroll 4
         for (uint32_t v = 0; v < row_v; ++v) {
             float kf[VN];
             Elem<T>::unpack(kv[v], kf);
@@ -159,6 +182,7 @@ __global__ void __launch_bounds__(LA_WARPS * 32) latent_split_kernel(const float
             for (int i = 0; i < NJ * VN; ++i) o[g][i] *= alpha;
         }
         const uint32_t nk = min((uint32_t)LA_KEYS, k1 - base);
+#pragma unroll 2
         for (uint32_t k = 0; k < nk; ++k) {
             float p[HG];
 #pragma unroll
@@ -199,47 +223,84 @@ __global__ void __launch_bounds__(LA_WARPS * 32) latent_split_kernel(const float
     }
 }
 
-// grid (slabs of a head's value rows, heads, queries): combine the splits with the sink, then this slab's rows of W_uv.
+// A cluster of four CTAs per (head, query): each combines the splits for a quarter of the latent's columns - the sink counts
+// in the denominator - and hands its quarter to the others through distributed shared memory; each then takes a quarter of
+// the head's rows of W_uv.
+constexpr uint32_t MERGE_CL = 4;
 template <class T>
-__global__ void __launch_bounds__(256) latent_merge_kernel(const float *part, LatentShape s, uint32_t splits, const float *__restrict__ sink,
-                                                           const float *gate, const T *__restrict__ uv, T *out, size_t ldo) {
+__global__ void __cluster_dims__(MERGE_CL, 1, 1) __launch_bounds__(256) latent_merge_kernel(const float *part, LatentShape s, uint32_t splits,
+                                                                                          const float *__restrict__ sink, const float *gate,
+                                                                                          const T *__restrict__ uv, T *out, size_t ldo) {
     extern __shared__ __align__(16) float lat[];  // [rank_p]
     __shared__ float wt[LATENT_MAX_SPLITS];
+    __shared__ float2 sums[4][64];
+    cg::cluster_group cluster = cg::this_cluster();
     pdl_trigger();
+    const uint32_t h = blockIdx.y, j = blockIdx.z, ps = s.rank_p + 2, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, cr = cluster.block_rank();
+    const uint32_t slab = (s.vdim_p + MERGE_CL - 1) / MERGE_CL, v0 = cr * slab, v1 = min(v0 + slab, s.vdim_p);
     pdl_wait();
-    const uint32_t h = blockIdx.y, j = blockIdx.z, ps = s.rank_p + 2, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const float *p = part + ((size_t)j * s.heads + h) * splits * ps;
     if (warp == 0) {
+        constexpr int PER = LATENT_MAX_SPLITS / 32;
         const float sk = sink[h];
-        float mx = sk;
-        for (uint32_t i = lane; i < splits; i += 32) mx = fmaxf(mx, p[(size_t)i * ps]);
+        float ms[PER], ls[PER], mx = sk;
+#pragma unroll
+        for (int i = 0; i < PER; ++i) {
+            const uint32_t sp = lane + 32 * i;
+            ms[i] = sp < splits ? p[(size_t)sp * ps] : -INFINITY;
+            ls[i] = sp < splits ? p[(size_t)sp * ps + 1] : 0.0f;
+            mx = fmaxf(mx, ms[i]);
+        }
         mx = warp_max(mx);
         float den = 0.0f;
-        for (uint32_t i = lane; i < splits; i += 32) {
-            const float e = expf(p[(size_t)i * ps] - mx);
-            wt[i] = e;
-            den += e * p[(size_t)i * ps + 1];
+#pragma unroll
+        for (int i = 0; i < PER; ++i) {
+            ms[i] = expf(ms[i] - mx);
+            den += ms[i] * ls[i];
         }
         den = warp_sum(den) + expf(sk - mx);
-        __syncwarp();
-        for (uint32_t i = lane; i < splits; i += 32) wt[i] /= den;
+#pragma unroll
+        for (int i = 0; i < PER; ++i)
+            if (lane + 32 * i < splits) wt[lane + 32 * i] = ms[i] / den;
     }
-    __syncthreads();
-    for (uint32_t c = threadIdx.x; c < s.rank_p; c += 256) {
-        float v = 0.0f;
+    cluster.sync();  // every CTA of the cluster runs before its shared memory is written from outside
+    const uint32_t quarter = s.rank_p / MERGE_CL, sub = threadIdx.x >> 6, tc = threadIdx.x & 63;  // rank_p is a multiple of 64
+    for (uint32_t c0 = 0; c0 < quarter; c0 += 128) {  // 64 threads x 2 columns, four of them share the splits
+        const uint32_t c = c0 + 2 * tc;
+        float2 a = make_float2(0.0f, 0.0f);
+        if (c < quarter) {
+            const float *src = p + 2 + cr * quarter + c;
 #pragma unroll 8
-        for (uint32_t i = 0; i < splits; ++i) v = fmaf(wt[i], p[(size_t)i * ps + 2 + c], v);
-        lat[c] = v;
+            for (uint32_t i = sub; i < splits; i += 4) {
+                const float2 v = *reinterpret_cast<const float2 *>(src + (size_t)i * ps);
+                a.x = fmaf(wt[i], v.x, a.x);
+                a.y = fmaf(wt[i], v.y, a.y);
+            }
+        }
+        sums[sub][tc] = a;
+        __syncthreads();
+        if (sub == 0 && c < quarter) {
+#pragma unroll
+            for (int i = 1; i < 4; ++i) {
+                a.x += sums[i][tc].x;
+                a.y += sums[i][tc].y;
+            }
+            sums[0][tc] = a;
+        }
+        __syncthreads();
+        // thread group `sub` writes the pair into CTA `sub` of the cluster
+        if (c < quarter) *reinterpret_cast<float2 *>(cluster.map_shared_rank(lat, sub) + cr * quarter + c) = sums[0][tc];
+        __syncthreads();
     }
-    __syncthreads();
+    cluster.sync();
     const float gt = gate[(size_t)j * s.heads + h];
-    const uint32_t slab = (s.vdim_p + gridDim.x - 1) / gridDim.x, v0 = blockIdx.x * slab, v1 = min(v0 + slab, s.vdim_p);
+#pragma unroll 4
     for (uint32_t v = v0 + warp; v < v1; v += 8) {
         const uint4 *w = reinterpret_cast<const uint4 *>(uv + ((size_t)h * s.vdim_p + v) * s.rank_p);
         float acc = 0.0f;
         for (uint32_t c = lane; c < s.rank_p / Elem<T>::N; c += 32) {
             float wf[Elem<T>::N];
-            Elem<T>::unpack(w[c], wf);
+            Elem<T>::unpack(__ldg(w + c), wf);
 #pragma unroll
             for (int i = 0; i < Elem<T>::N; ++i) acc = fmaf(wf[i], lat[c * Elem<T>::N + i], acc);
         }
@@ -282,9 +343,8 @@ int32_t latent_attention(const float *q32, const LatentShape &s, const void *uk,
         return fail(CERA_CUDA_ERR_UNSUPPORTED, "latent attention: rank %u", s.rank);
     };
     CERA_TRY(few ? split(std::integral_constant<int, 1>{}) : split(std::integral_constant<int, 4>{}));
-    const uint32_t slabs = n == 1 ? 4 : 1;
     count_launch();
-    return check_cuda(launch_k(latent_merge_kernel<T>, dim3(slabs, s.heads, (unsigned)n), dim3(256), (size_t)s.rank_p * 4, st, (const float *)ws.part, s, splits,
+    return check_cuda(launch_k(latent_merge_kernel<T>, dim3(MERGE_CL, s.heads, (unsigned)n), dim3(256), (size_t)s.rank_p * 4, st, (const float *)ws.part, s, splits,
                                sink, gate, (const T *)uv, (T *)out, ldo),
                       "latent merge launch");
 }
@@ -293,7 +353,7 @@ int32_t latent_attention(const float *q32, const LatentShape &s, const void *uk,
 
 uint32_t latent_splits(size_t n_positions) {
     uint32_t s = 1;
-    while (s < LATENT_MAX_SPLITS && s * 64 < n_positions) s *= 2;
+    while (s < LATENT_MAX_SPLITS && s * LA_KEYS < n_positions) s *= 2;
     return s;
 }
 

@@ -6,8 +6,8 @@ namespace cera {
 
 namespace {
 
-// One CTA per T tokens.  Warps take experts round-robin; lane-strided f32 dots (a router element is loaded once for the T
-// tokens), shuffle tree; then warp t picks for token t.
+// One CTA per T tokens.  A warp takes four experts at a time: lane-strided float4 dots in f32, every router and token
+// vector loaded once for the 4 T products it enters; shuffle tree; then warp t picks for token t.
 template <int T>
 __global__ void __launch_bounds__(256) moe_route_kernel(const float *x, const float *__restrict__ router,
                                                         const float *__restrict__ bias, uint32_t hidden, uint32_t ld_x, uint32_t n, uint32_t n_expert,
@@ -23,19 +23,31 @@ __global__ void __launch_bounds__(256) moe_route_kernel(const float *x, const fl
     const float *xj[T];
 #pragma unroll
     for (int t = 0; t < T; ++t) xj[t] = x + (size_t)min(j0 + t, n - 1) * ld_x;
-    for (uint32_t e = warp; e < n_expert; e += blockDim.x >> 5) {
-        const float *r = router + (size_t)e * hidden;
-        float acc[T] = {};
-        for (uint32_t i = lane; i < hidden; i += 32) {
-            const float rv = r[i];
+    constexpr int EG = 4;
+    for (uint32_t e0 = warp * EG; e0 < n_expert; e0 += (blockDim.x >> 5) * EG) {
+        const float4 *r[EG];
 #pragma unroll
-            for (int t = 0; t < T; ++t) acc[t] = fmaf(rv, xj[t][i], acc[t]);
+        for (int g = 0; g < EG; ++g) r[g] = reinterpret_cast<const float4 *>(router + (size_t)min(e0 + g, n_expert - 1) * hidden);
+        float acc[EG][T] = {};
+        for (uint32_t i = lane; i < hidden / 4; i += 32) {
+            float4 rv[EG];
+#pragma unroll
+            for (int g = 0; g < EG; ++g) rv[g] = __ldg(r[g] + i);
+#pragma unroll
+            for (int t = 0; t < T; ++t) {
+                const float4 xv = reinterpret_cast<const float4 *>(xj[t])[i];
+#pragma unroll
+                for (int g = 0; g < EG; ++g)
+                    acc[g][t] = fmaf(rv[g].w, xv.w, fmaf(rv[g].z, xv.z, fmaf(rv[g].y, xv.y, fmaf(rv[g].x, xv.x, acc[g][t]))));
+            }
         }
 #pragma unroll
-        for (int t = 0; t < T; ++t) {
-            acc[t] = warp_sum(acc[t]);
-            if (lane == 0) probs[t][e] = acc[t];
-        }
+        for (int g = 0; g < EG; ++g)
+#pragma unroll
+            for (int t = 0; t < T; ++t) {
+                const float v = warp_sum(acc[g][t]);
+                if (lane == 0 && e0 + g < n_expert) probs[t][e0 + g] = v;
+            }
     }
     __syncthreads();
 #pragma unroll 1
