@@ -145,7 +145,7 @@ int32_t launch_latent_prepare(const float *in, const LatentShape &s, size_t n, s
 // Attention in the latent space for n queries at positions start_pos + j (or *len_dev - 1): q_lat = W_uk^T q, scores
 // against the cached latents, per-split partial sums, merge with the sink, W_uv, gate.  out [n][ldo] of T, heads * vdim_p used.
 struct LatentScratch {
-    float *q_lat = nullptr;  // [queries][heads][rank_p + rot_p]
+    float *q_lat = nullptr;  // [queries][heads][rank_p + rot_p] f32, or as many pairs of bf16
     float *part = nullptr;   // [queries][heads][splits][rank_p + 2]
 };
 constexpr uint32_t LATENT_MAX_SPLITS = 128;  // queries * splits of one call never exceed this

@@ -50,7 +50,8 @@ __global__ void __launch_bounds__(256) latent_prepare_kernel(const float *in, La
     }
 }
 
-// q_lat[j][h] = [W_uk_h^T q_h, rotated part].  grid (64-column slabs of rank_p, heads, queries), 256 threads = 16 slices of
+// [W_uk_h^T q_h, rotated part] of every (query, head): f32, or for the tensor cores a bf16 high part and the bf16 of what it
+// leaves (16 bits of the query survive; the low parts follow all the high parts).  grid (64-column slabs of rank_p, heads, queries), 256 threads = 16 slices of
 // the head's dimensions x 16 groups of four columns; weights are fetched ahead of the wait.
 template <class T>
 __global__ void __launch_bounds__(256) latent_query_kernel(const float *q32, LatentShape s, const T *__restrict__ uk, float *q_lat) {
@@ -84,20 +85,30 @@ __global__ void __launch_bounds__(256) latent_query_kernel(const float *q32, Lat
     for (uint32_t d = sl + 16 * PRE; d < s.dim_p; d += 16) add(*reinterpret_cast<const V *>(w + (size_t)d * s.rank_p), q[d]);
     part[sl][cg] = acc;
     __syncthreads();
-    float *o = q_lat + ((size_t)j * s.heads + h) * ldo;
+    const size_t at = ((size_t)j * s.heads + h) * ldo, low = (size_t)gridDim.z * s.heads * ldo;
+    auto put = [&](uint32_t i, float v) {
+        if constexpr (sizeof(T) == 4) {
+            q_lat[at + i] = v;
+        } else {
+            bf16 *o = reinterpret_cast<bf16 *>(q_lat);
+            const bf16 hi = __float2bfloat16_rn(v);
+            o[at + i] = hi;
+            o[low + at + i] = __float2bfloat16_rn(v - __bfloat162float(hi));
+        }
+    };
     if (threadIdx.x < 64) {
         float v = 0.0f;
 #pragma unroll
         for (int i = 0; i < 16; ++i) v += reinterpret_cast<const float *>(part[i])[threadIdx.x];
-        o[blockIdx.x * 64 + threadIdx.x] = v;
+        put(blockIdx.x * 64 + threadIdx.x, v);
     } else if (blockIdx.x == 0) {
-        for (uint32_t i = threadIdx.x - 64; i < s.rot_p; i += 192) o[s.rank_p + i] = q[s.dim_p + i];
+        for (uint32_t i = threadIdx.x - 64; i < s.rot_p; i += 192) put(s.rank_p + i, q[s.dim_p + i]);
     }
 }
 
 constexpr int LA_WARPS = 4, LA_KEYS = 32;
 
-// One CTA: (split of the keys, 4 HG heads, query).  Tiles of 32 keys in shared memory; a warp owns HG heads: scores with
+// The f32 form.  One CTA: (split of the keys, 4 HG heads, query).  Tiles of 32 keys in shared memory; a warp owns HG heads: scores with
 // lane = key, online softmax, weighted latents with lane = columns.
 template <class T, int HG, int NJ>
 __global__ void __launch_bounds__(LA_WARPS * 32) latent_split_kernel(const float *q_lat, LatentShape s, const T *cache_c, const T *cache_r, uint32_t start_pos,
@@ -223,6 +234,200 @@ __global__ void __launch_bounds__(LA_WARPS * 32) latent_split_kernel(const float
     }
 }
 
+// ---- the bf16 form on mma.sync: 16 heads are one operand tile ------------------------------------------------------------
+// One CTA: (split of the keys, 16 heads, query); tiles of 64 keys.  Scores: warp = 16 keys, the query as a high and a low
+// bf16 part (two products into one f32 accumulator).  Softmax in f32 over the CTA's tile; the weights enter the second
+// product as a high and a low part as well.  Weighted latents: warp = a quarter of the latent's columns, NP pairs of 8.
+constexpr int LM_KEYS = 64, LM_HEADS = 16, LM_P_LD = LM_KEYS + 8;
+
+__device__ __forceinline__ void ldsm4(uint32_t (&r)[4], const void *p) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(tma::smem_u32(p)) : "memory");
+}
+__device__ __forceinline__ void ldsm4_trans(uint32_t (&r)[4], const void *p) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(tma::smem_u32(p)) : "memory");
+}
+__device__ __forceinline__ void mma_bf16(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+
+template <int NP>
+__global__ void __launch_bounds__(128) latent_split_mma_kernel(const bf16 *q, LatentShape s, const bf16 *cache_c, const bf16 *cache_r, uint32_t start_pos,
+                                                              const uint32_t *len_dev, uint32_t splits, int stages, float *part) {
+    extern __shared__ __align__(16) uint8_t smem[];
+    __shared__ float row_max[4][LM_HEADS], row_sum[4][LM_HEADS];
+    __shared__ __align__(16) bf16 pw[2][LM_HEADS][LM_P_LD];  // weights of the tile: high, low
+    pdl_trigger();
+    const uint32_t ql = s.rank_p + s.rot_p, ld = ql + 8, row_v = ql / 8, c_v = s.rank_p / 8;
+    bf16 *qs = reinterpret_cast<bf16 *>(smem), *tile = qs + 2 * LM_HEADS * ld;  // qs: [high, low][16][ld]
+    const uint32_t split = blockIdx.x, h0 = blockIdx.y * LM_HEADS, j = blockIdx.z, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    pdl_wait();
+    const uint32_t len = len_dev ? *len_dev : start_pos + j + 1;
+    const uint32_t per = ((len + splits - 1) / splits + LM_KEYS - 1) / LM_KEYS * LM_KEYS, k0 = min(split * per, len), k1 = min(k0 + per, len);
+    const size_t low = (size_t)gridDim.z * s.heads * ql;
+    for (uint32_t r = warp; r < 2 * LM_HEADS; r += 4) {
+        const uint32_t h = h0 + (r & 15);
+        const bf16 *src = q + (r >> 4) * low + ((size_t)j * s.heads + h) * ql;
+        for (uint32_t v = lane; v < row_v; v += 32) {
+            if (h < s.heads) tma::cp_async16(qs + (size_t)r * ld + v * 8, src + v * 8);
+            else *reinterpret_cast<uint4 *>(qs + (size_t)r * ld + v * 8) = make_uint4(0, 0, 0, 0);
+        }
+    }
+    auto fetch = [&](uint32_t base, int stage) {
+        bf16 *dst = tile + (size_t)stage * LM_KEYS * ld;
+        for (uint32_t k = warp; k < LM_KEYS; k += 4) {
+            const bf16 *cr = cache_c + (size_t)(base + k) * s.rank_p, *rr = cache_r + (size_t)(base + k) * s.rot_p;
+            for (uint32_t v = lane; v < row_v; v += 32) {
+                if (base + k < k1) tma::cp_async16(dst + (size_t)k * ld + v * 8, v < c_v ? cr + v * 8 : rr + (v - c_v) * 8);
+                else *reinterpret_cast<uint4 *>(dst + (size_t)k * ld + v * 8) = make_uint4(0, 0, 0, 0);
+            }
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    float o[NP][2][4], m[2] = {-INFINITY, -INFINITY}, l[2] = {0.0f, 0.0f};  // rows lane / 4 and lane / 4 + 8
+#pragma unroll
+    for (int i = 0; i < NP; ++i)
+#pragma unroll
+        for (int n = 0; n < 2; ++n)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) o[i][n][e] = 0.0f;
+    const uint32_t r0 = lane >> 2, col2 = (lane & 3) * 2, cols = s.rank_p / 4, c_base = warp * cols;  // cols: a multiple of 16
+    const float sc2 = s.scale * 1.44269504088896340736f;
+    int stage = 0;
+    if (k0 < k1) fetch(k0, 0);
+    for (uint32_t base = k0; base < k1; base += LM_KEYS) {
+        const bool more = base + LM_KEYS < k1 && stages == 2;
+        if (more) fetch(base + LM_KEYS, stage ^ 1);
+        if (more) asm volatile("cp.async.wait_group 1;" ::: "memory");
+        else asm volatile("cp.async.wait_group 0;" ::: "memory");
+        __syncthreads();
+        const bf16 *tl = tile + (size_t)stage * LM_KEYS * ld;
+        float sc[2][4] = {};
+        {
+            const bf16 *qa = qs + (size_t)(lane & 15) * ld + (lane >> 4) * 8;
+            const bf16 *kb = tl + (size_t)(warp * 16 + (lane & 7) + (lane >> 4) * 8) * ld + ((lane >> 3) & 1) * 8;
+#pragma unroll 4
+            for (uint32_t k = 0; k < ql; k += 16) {
+                uint32_t ah[4], al[4], b[4];
+                ldsm4(ah, qa + k);
+                ldsm4(al, qa + (size_t)LM_HEADS * ld + k);
+                ldsm4(b, kb + k);
+                mma_bf16(sc[0], ah, b[0], b[1]);
+                mma_bf16(sc[1], ah, b[2], b[3]);
+                mma_bf16(sc[0], al, b[0], b[1]);
+                mma_bf16(sc[1], al, b[2], b[3]);
+            }
+        }
+        float mx[2] = {-INFINITY, -INFINITY};
+#pragma unroll
+        for (int n = 0; n < 2; ++n)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                const uint32_t key = base + warp * 16 + n * 8 + col2 + (e & 1);
+                sc[n][e] = key < k1 ? sc[n][e] * sc2 : -INFINITY;
+                mx[e >> 1] = fmaxf(mx[e >> 1], sc[n][e]);
+            }
+#pragma unroll
+        for (int r = 0; r < 2; ++r) {
+            mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 1));
+            mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 2));
+            if ((lane & 3) == 0) row_max[warp][r0 + 8 * r] = mx[r];
+        }
+        __syncthreads();
+        float alpha[2];
+#pragma unroll
+        for (int r = 0; r < 2; ++r) {
+            const uint32_t row = r0 + 8 * r;
+            // the first key of a tile is always valid: the maximum is finite
+            const float mn = fmaxf(m[r], fmaxf(fmaxf(row_max[0][row], row_max[1][row]), fmaxf(row_max[2][row], row_max[3][row])));
+            alpha[r] = exp2f(m[r] - mn);
+            m[r] = mn;
+            l[r] *= alpha[r];
+        }
+#pragma unroll
+        for (int n = 0; n < 2; ++n)
+#pragma unroll
+            for (int r = 0; r < 2; ++r) {
+                const float e0 = exp2f(sc[n][2 * r] - m[r]), e1 = exp2f(sc[n][2 * r + 1] - m[r]);
+                l[r] += e0 + e1;
+                const __nv_bfloat162 hi = __floats2bfloat162_rn(e0, e1);
+                const float2 hf = __bfloat1622float2(hi);
+                const uint32_t c = warp * 16 + n * 8 + col2;
+                *reinterpret_cast<__nv_bfloat162 *>(&pw[0][r0 + 8 * r][c]) = hi;
+                *reinterpret_cast<__nv_bfloat162 *>(&pw[1][r0 + 8 * r][c]) = __floats2bfloat162_rn(e0 - hf.x, e1 - hf.y);
+            }
+#pragma unroll
+        for (int i = 0; i < NP; ++i)
+#pragma unroll
+            for (int n = 0; n < 2; ++n)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) o[i][n][e] *= alpha[e >> 1];
+        __syncthreads();
+        const bf16 *vb = tl + (size_t)((lane & 7) + ((lane >> 3) & 1) * 8) * ld + c_base + (lane >> 4) * 8;
+#pragma unroll 1
+        for (uint32_t k = 0; k < LM_KEYS; k += 16) {
+            uint32_t ph[4], pl[4];
+            ldsm4(ph, &pw[0][lane & 15][k + (lane >> 4) * 8]);
+            ldsm4(pl, &pw[1][lane & 15][k + (lane >> 4) * 8]);
+#pragma unroll
+            for (int i = 0; i < NP; ++i)
+                if ((uint32_t)i * 16 < cols) {
+                    uint32_t b[4];
+                    ldsm4_trans(b, vb + (size_t)k * ld + i * 16);
+                    mma_bf16(o[i][0], ph, b[0], b[1]);
+                    mma_bf16(o[i][1], ph, b[2], b[3]);
+                    mma_bf16(o[i][0], pl, b[0], b[1]);
+                    mma_bf16(o[i][1], pl, b[2], b[3]);
+                }
+        }
+        __syncthreads();
+        if (stages == 2) stage ^= 1;
+        else if (base + LM_KEYS < k1) fetch(base + LM_KEYS, 0);
+    }
+    // per row: maximum (natural units), sum of weights over the four warps' keys, weighted latents
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+        l[r] += __shfl_xor_sync(0xffffffffu, l[r], 1);
+        l[r] += __shfl_xor_sync(0xffffffffu, l[r], 2);
+        if ((lane & 3) == 0) row_sum[warp][r0 + 8 * r] = l[r];
+    }
+    asm volatile("cp.async.wait_all;" ::: "memory");  // a split without keys has still asked for its queries
+    __syncthreads();
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+        const uint32_t row = r0 + 8 * r, h = h0 + row;
+        if (h >= s.heads) continue;
+        float *po = part + (((size_t)j * s.heads + h) * splits + split) * (s.rank_p + 2);
+        if (warp == 0 && (lane & 3) == 0) {
+            po[0] = m[r] * 0.69314718055994530942f;
+            po[1] = row_sum[0][row] + row_sum[1][row] + row_sum[2][row] + row_sum[3][row];
+        }
+#pragma unroll
+        for (int i = 0; i < NP; ++i)
+            if ((uint32_t)i * 16 < cols) {
+#pragma unroll
+                for (int n = 0; n < 2; ++n)
+                    *reinterpret_cast<float2 *>(po + 2 + c_base + i * 16 + n * 8 + col2) = make_float2(o[i][n][2 * r], o[i][n][2 * r + 1]);
+            }
+    }
+}
+
+template <int NP>
+int32_t launch_split_mma(const LatentScratch &ws, const LatentShape &s, const void *cc, const void *cr, size_t n, size_t start_pos, const uint32_t *len_dev,
+                         uint32_t splits, cudaStream_t st) {
+    const size_t ld = s.rank_p + s.rot_p + 8, qb = 2 * LM_HEADS * ld * 2, tb = LM_KEYS * ld * 2;
+    const int stages = qb + 2 * tb <= 215 * 1024 ? 2 : 1;
+    const size_t bytes = qb + stages * tb;
+    if (bytes > 215 * 1024) return fail(CERA_CUDA_ERR_UNSUPPORTED, "latent attention: rank %u with %u rotated dimensions", s.rank, s.rot);
+    auto k = latent_split_mma_kernel<NP>;
+    CERA_CUDA_TRY(cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, 215 * 1024));
+    count_launch();
+    return check_cuda(launch_k(k, dim3(splits, (s.heads + LM_HEADS - 1) / LM_HEADS, (unsigned)n), dim3(128), bytes, st, (const bf16 *)ws.q_lat, s, (const bf16 *)cc,
+                               (const bf16 *)cr, (uint32_t)start_pos, len_dev, splits, stages, ws.part),
+                      "latent split launch");
+}
+
 // A cluster of four CTAs per (head, query): each combines the splits for a quarter of the latent's columns - the sink counts
 // in the denominator - and hands its quarter to the others through distributed shared memory; each then takes a quarter of
 // the head's rows of W_uv.
@@ -331,18 +536,23 @@ int32_t latent_attention(const float *q32, const LatentShape &s, const void *uk,
                          size_t ldo, cudaStream_t st) {
     count_launch();
     CERA_CUDA_TRY(launch_k(latent_query_kernel<T>, dim3(s.rank_p / 64, s.heads, (unsigned)n), dim3(256), 0, st, q32, s, (const T *)uk, ws.q_lat));
-    const uint32_t nj = (s.rank_p / Elem<T>::N + 31) / 32;
-    const bool few = s.heads <= 8;  // one head per warp
-    auto split = [&](auto hg) -> int32_t {
-        constexpr int HG = decltype(hg)::value;
-        if (nj <= 1) return launch_split<T, HG, 1>(ws, s, cc, cr, n, start_pos, len_dev, splits, st);
-        if (nj <= 2) return launch_split<T, HG, 2>(ws, s, cc, cr, n, start_pos, len_dev, splits, st);
-        if (nj <= 4) return launch_split<T, HG, 4>(ws, s, cc, cr, n, start_pos, len_dev, splits, st);
-        if constexpr (Elem<T>::N == 4)
-            if (nj <= 8) return launch_split<T, HG, 8>(ws, s, cc, cr, n, start_pos, len_dev, splits, st);
-        return fail(CERA_CUDA_ERR_UNSUPPORTED, "latent attention: rank %u", s.rank);
-    };
-    CERA_TRY(few ? split(std::integral_constant<int, 1>{}) : split(std::integral_constant<int, 4>{}));
+    int32_t rc;
+    if constexpr (sizeof(T) == 2) {
+        rc = s.rank_p <= 256   ? launch_split_mma<4>(ws, s, cc, cr, n, start_pos, len_dev, splits, st)
+             : s.rank_p <= 512 ? launch_split_mma<8>(ws, s, cc, cr, n, start_pos, len_dev, splits, st)
+                               : launch_split_mma<16>(ws, s, cc, cr, n, start_pos, len_dev, splits, st);
+    } else {
+        const uint32_t nj = (s.rank_p / 4 + 31) / 32;
+        auto split = [&](auto hg) -> int32_t {
+            constexpr int HG = decltype(hg)::value;
+            if (nj <= 1) return launch_split<T, HG, 1>(ws, s, cc, cr, n, start_pos, len_dev, splits, st);
+            if (nj <= 2) return launch_split<T, HG, 2>(ws, s, cc, cr, n, start_pos, len_dev, splits, st);
+            if (nj <= 4) return launch_split<T, HG, 4>(ws, s, cc, cr, n, start_pos, len_dev, splits, st);
+            return launch_split<T, HG, 8>(ws, s, cc, cr, n, start_pos, len_dev, splits, st);
+        };
+        rc = s.heads <= 8 ? split(std::integral_constant<int, 1>{}) : split(std::integral_constant<int, 4>{});  // few heads: one per warp
+    }
+    CERA_TRY(rc);
     count_launch();
     return check_cuda(launch_k(latent_merge_kernel<T>, dim3(MERGE_CL, s.heads, (unsigned)n), dim3(256), (size_t)s.rank_p * 4, st, (const float *)ws.part, s, splits,
                                sink, gate, (const T *)uv, (T *)out, ldo),
@@ -353,7 +563,7 @@ int32_t latent_attention(const float *q32, const LatentShape &s, const void *uk,
 
 uint32_t latent_splits(size_t n_positions) {
     uint32_t s = 1;
-    while (s < LATENT_MAX_SPLITS && s * LA_KEYS < n_positions) s *= 2;
+    while (s < LATENT_MAX_SPLITS && s * LM_KEYS < n_positions) s *= 2;
     return s;
 }
 
