@@ -543,7 +543,7 @@ def cuda_arm(args, rank, world):
     e2e_toks = []
     t0 = time.perf_counter()
     for _ in range(K):
-        tok = model.forward_greedy(tok, pos)  # 16 bytes in (token, pos, len, step), 4 bytes out
+        tok = model.forward_greedy(tok, pos)  # 20 bytes in (token, pos, len, step, previous token), 4 bytes out
         e2e_toks.append(tok)
         pos += 1
     e2e_s = time.perf_counter() - t0
@@ -591,7 +591,7 @@ def cuda_arm(args, rank, world):
             "prompt": {"batched_prefill_s": round(t_pre, 4), "batched_prefill_tok_s": round(prompt_len / t_pre, 1),
                        "per_token_prefill_s": round(t_pt, 3), "build_s": round(t_build, 2)},
             "stream_check": stream_check,
-            "e2e": {"value": K / e2e_s, "unit": UNIT, "h2d_bytes_per_step": 12, "d2h_bytes_per_step": 4},
+            "e2e": {"value": K / e2e_s, "unit": UNIT, "h2d_bytes_per_step": 20, "d2h_bytes_per_step": 4},
             "gpu_launches": int(model_launches + roof_launches),
             "gpu_launches_per_rank": per_rank_launches,  # the model's kernels in the timed regions, by rank (rank 0 also runs the kernel microbench)
             "clocks": clocks,

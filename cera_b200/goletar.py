@@ -31,7 +31,7 @@ def _layer(i, entry):
         d.recurrent_width = m["width"]
     else:
         raise ValueError(f"layer {i}: unknown mixer {entry['type']!r}")
-    mlp = entry["mlp"]
+    mlp = entry.get("mlp")
     if mlp is None:
         d.ff = Ff.NONE
     elif mlp["kind"] == "moe":

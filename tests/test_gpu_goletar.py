@@ -334,3 +334,50 @@ def test_no_bounded_wait_ran_out():
     need_gpu()
     from cera_b200 import _lib
     assert _lib.kernel_status() == 0
+
+
+def moe_by_rule(h, w, c, softmax, renorm, weight_input):
+    """The plain routed feed-forward under the other rules a layer description can name."""
+    z = h @ w["router"].T
+    s = np.exp(z - z.max(-1, keepdims=True)) if softmax else G.sigmoid(z)
+    if softmax:
+        s /= s.sum(-1, keepdims=True)
+    out = np.zeros_like(h)
+    for t in range(len(h)):
+        ids = np.argsort(-s[t], kind="stable")[:c["router"]["top"]]
+        wt = s[t][ids] / (s[t][ids].sum() if renorm else 1.0)
+        for e, x in zip(ids, wt):
+            m = (w[f"e{e}.gate"], w[f"e{e}.up"], w[f"e{e}.down"], c["expert"]["limit"])
+            out[t] += G.clamped_glu(x * h[t], *m) if weight_input else x * G.clamped_glu(h[t], *m)
+    return out
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("rule", [(1, 0, 1), (0, 1, 0), (1, 1, 0)])
+def test_other_rules_of_a_layer_description(monkeypatch, dtype, rule):
+    """Softmax scores, renormalised weights, weights on the output, per-channel norms: the mechanisms' parameters, not this design's."""
+    need_gpu()
+    from cera_b200 import goletar
+    from cera_b200.layered import LayeredModel
+    from cera_b200.types import BF16
+    softmax, renorm, weight_input = rule
+    cfg = config([attention(mlp=moe(experts=3, top=3)), mingru(mlp=moe(experts=4, top=4, ff=72))])
+    w = G.random_weights(cfg, 111)
+    rng = np.random.default_rng(112)
+    for name in ("l0.norm1", "l0.norm1b", "l1.norm2", "l1.norm2b", "final.norm"):
+        w[name] = G.from_bf16(G.to_bf16(1.0 + 0.3 * rng.standard_normal(72))).astype(np.float64)
+    kw, layers = goletar.describe(cfg)
+    for d in layers:
+        d.router_softmax, d.router_renorm, d.weight_input = softmax, renorm, weight_input
+    m = LayeredModel(layers, dtype=dtype, max_seq_len=120, **kw)
+    for name, role, layer, expert in goletar.tensor_roles(layers):
+        v = w[name]
+        rows, cols = v.shape if v.ndim == 2 else (1, v.size)
+        m.add_tensor(role, layer, BF16, rows, cols, G.to_bf16(v).reshape(-1), expert=expert)
+    m.finalize()
+    monkeypatch.setattr(G, "moe", lambda h, ww, c: moe_by_rule(h, ww, c, *rule))
+    toks = tokens(110, cfg["vocab"], 113)
+    want = G.logits(toks, cfg, w)
+    for sizes in ([110], [50, 1]):
+        assert error(feed(m, toks, sizes), want) < TOL[dtype], sizes
+    m.close()
