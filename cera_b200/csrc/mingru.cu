@@ -1,5 +1,5 @@
-// minGRU over a prompt portion: S_t = (1 - z_t) S_(t-1) + z_t candidate_t per element, gates read from the current token
-// only, so a portion is a linear scan.  A CTA owns 32 elements; its warps cut the portion into segments, each warp
+// minGRU over a prompt portion: S_t = (1 - z_t) S_(t-1) + z_t candidate_t per element.  z and the candidate depend on
+// token t alone, which makes a portion a linear scan.  A CTA owns 32 elements; its warps cut the portion into segments, each warp
 // composes its segment into one affine map (A, B), the maps are combined in shared memory, and every warp then walks its
 // segment from the state it starts in.  f32 throughout.
 #include "dense.cuh"

@@ -293,8 +293,8 @@ typedef struct {
     int32_t ff;
     /* latent attention: per head head_dim unrotated and rot_dim rotated query / key dimensions; keys and values are
      * up-projections of one normed latent of kv_rank numbers per position, the rotated key part is shared by all heads.
-     * Adjacent dimensions rotate in pairs by pos * rope_base^(-2i / rot_dim).  The softmax denominator also holds
-     * exp(sink) per head; each head's output is multiplied by sigmoid(gate). */
+     * Adjacent dimensions rotate in pairs by pos * rope_base^(-2i / rot_dim).  Per head a sink joins the
+     * softmax denominator as exp(sink), and sigmoid(gate) scales the result. */
     uint32_t n_heads, head_dim, rot_dim, value_dim, kv_rank;
     float rope_base, attn_scale;
     /* gated recurrence: S = (1 - z) S + z candidate, per element, recurrent_width elements */
