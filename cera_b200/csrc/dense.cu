@@ -15,19 +15,19 @@ __device__ __forceinline__ float load_src(const void *p, int type, size_t i) {
 }
 
 __global__ void place_kernel(const void *__restrict__ src, int type, size_t rows, uint32_t cols, void *dst, int dst_f32, size_t ld, PadMap rmap,
-                             PadMap cmap) {
+                             PadMap cmap, float offset) {
     const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
     if (i >= rows * cols) return;
     const uint32_t r = (uint32_t)(i / cols), c = (uint32_t)(i - (size_t)r * cols);
     const size_t o = (size_t)rmap(r) * ld + cmap(c);
-    const float v = load_src(src, type, i);
+    const float v = load_src(src, type, i) + offset;
     if (dst_f32) ((float *)dst)[o] = v;
     else ((bf16 *)dst)[o] = __float2bfloat16_rn(v);
 }
 
 template <class T>
 __global__ void __launch_bounds__(256) embed_dense_kernel(const T *__restrict__ table, const T *__restrict__ bigram, BigramParams bp, uint32_t ld,
-                                                          const uint32_t *tokens, const uint32_t *dyn, float *x) {
+                                                          const uint32_t *tokens, const uint32_t *dyn, float scale, float *x, float *keep) {
     pdl_trigger();
     pdl_wait();
     const uint32_t j = blockIdx.y;
@@ -39,9 +39,10 @@ __global__ void __launch_bounds__(256) embed_dense_kernel(const T *__restrict__ 
         brow = bigram + (size_t)b * ld;
     }
     for (uint32_t i = blockIdx.x * blockDim.x + threadIdx.x; i < ld; i += gridDim.x * blockDim.x) {
-        float v = Elem<T>::to(row[i]);
+        float v = Elem<T>::to(row[i]) * scale;
         if (brow) v += Elem<T>::to(brow[i]);
         x[(size_t)j * ld + i] = v;
+        if (keep) keep[(size_t)j * ld + i] = v;
     }
 }
 
@@ -82,22 +83,39 @@ __global__ void __launch_bounds__(1024) residual_norm_kernel(ResidualNorm p, uin
                     }
             }
         }
+        float r = 1.0f;
+        if (p.post.g) {
 #pragma unroll
-        for (int e = 0; e < V; ++e) ss += yv[e].x * yv[e].x + yv[e].y * yv[e].y + yv[e].z * yv[e].z + yv[e].w * yv[e].w;
-        const float r = 1.0f / sqrtf(cta_sum(ss, red) * inv_w + eps);
+            for (int e = 0; e < V; ++e) ss += yv[e].x * yv[e].x + yv[e].y * yv[e].y + yv[e].z * yv[e].z + yv[e].w * yv[e].w;
+            r = 1.0f / sqrtf(cta_sum(ss, red) * inv_w + eps);
+        }
 #pragma unroll
         for (int e = 0; e < V; ++e) {
             const uint32_t i = t + e * nt;
             if (i < nv) {
-                const float4 g = p.post.at(i);
+                const float4 g = p.post.g ? p.post.at(i) : make_float4(1.0f, 1.0f, 1.0f, 1.0f);
                 xv[e].x += yv[e].x * r * g.x;
                 xv[e].y += yv[e].y * r * g.y;
                 xv[e].z += yv[e].z * r * g.z;
                 xv[e].w += yv[e].w * r * g.w;
-                x[i] = xv[e];
             }
         }
         ss = 0.0f;
+    }
+    if (p.y || p.add) {
+#pragma unroll
+        for (int e = 0; e < V; ++e) {
+            const uint32_t i = t + e * nt;
+            if (i >= nv) continue;
+            if (p.add) {
+                const float4 a = reinterpret_cast<const float4 *>(p.add + (size_t)j * ld)[i];
+                xv[e].x += a.x;
+                xv[e].y += a.y;
+                xv[e].z += a.z;
+                xv[e].w += a.w;
+            }
+            x[i] = xv[e];
+        }
     }
 #pragma unroll
     for (int e = 0; e < V; ++e) ss += xv[e].x * xv[e].x + xv[e].y * xv[e].y + xv[e].z * xv[e].z + xv[e].w * xv[e].w;
@@ -134,26 +152,26 @@ __global__ void __launch_bounds__(128) moe_gather_kernel(const uint4 *h, uint32_
 }  // namespace
 
 int32_t launch_place(const void *src, int32_t src_type, size_t rows, size_t cols, void *dst, int dst_f32, size_t ld, const PadMap &rmap,
-                     const PadMap &cmap, cudaStream_t st) {
+                     const PadMap &cmap, cudaStream_t st, float offset) {
     if (src_type != CERA_TYPE_F32 && src_type != CERA_TYPE_F16 && src_type != CERA_TYPE_BF16)
         return fail(CERA_CUDA_ERR_UNSUPPORTED, "dense weight: ggml type %d is not F32, F16 or BF16", src_type);
     const size_t total = rows * cols;
     if (total == 0) return CERA_CUDA_OK;
-    place_kernel<<<(unsigned)((total + 255) / 256), 256, 0, st>>>(src, src_type, rows, (uint32_t)cols, dst, dst_f32, ld, rmap, cmap);
+    place_kernel<<<(unsigned)((total + 255) / 256), 256, 0, st>>>(src, src_type, rows, (uint32_t)cols, dst, dst_f32, ld, rmap, cmap, offset);
     count_launch();
     return check_cuda(cudaGetLastError(), "place launch");
 }
 
 int32_t launch_embed_dense(const DenseView &table, const DenseView &bigram, const BigramParams &bp, const uint32_t *tokens, const uint32_t *dyn,
-                           size_t n, float *x, cudaStream_t st) {
+                           size_t n, float scale, float *x, float *keep, cudaStream_t st) {
     if (n == 0) return CERA_CUDA_OK;
     const dim3 grid((table.ld + 1023) / 1024, (unsigned)n);
     count_launch();
     if (table.f32)
         return check_cuda(launch_k(embed_dense_kernel<float>, grid, dim3(256), 0, st, (const float *)table.w, (const float *)bigram.w, bp, table.ld,
-                                   tokens, dyn, x), "embed launch");
+                                   tokens, dyn, scale, x, keep), "embed launch");
     return check_cuda(launch_k(embed_dense_kernel<bf16>, grid, dim3(256), 0, st, (const bf16 *)table.w, (const bf16 *)bigram.w, bp, table.ld, tokens,
-                               dyn, x), "embed launch");
+                               dyn, scale, x, keep), "embed launch");
 }
 
 int32_t launch_residual_norm(const ResidualNorm &p, uint32_t width, uint32_t ld, size_t n, float eps, cudaStream_t st) {

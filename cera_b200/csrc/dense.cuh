@@ -44,6 +44,7 @@ __device__ __forceinline__ void store4(bf16 *p, const float4 &v) {
 
 __device__ __forceinline__ float sigmoid_f32(float x) { return __fdividef(1.0f, 1.0f + expf(-x)); }
 __device__ __forceinline__ float silu_f32(float x) { return x * sigmoid_f32(x); }
+__device__ __forceinline__ float softplus_f32(float x) { return x > 20.0f ? x : log1pf(expf(x)); }
 // min(g, limit) * sigmoid(alpha g) * (clamp(u) + shift)
 __device__ __forceinline__ float gated_unit(float g, float u, const ExpertAct &a) {
     g = fminf(g, a.limit);

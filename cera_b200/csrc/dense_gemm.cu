@@ -24,15 +24,15 @@ __global__ void __launch_bounds__(256) dense_gemm_kernel(DenseGemm g) {
         end = t.first + t.count;
         if (first >= end) return;
     }
-    const uint32_t r0 = blockIdx.x * GM_TILE, ld = g.w.ld;
-    const T *w = (const T *)g.w.w + (size_t)row_base * ld, *x = (const T *)g.x;
+    const uint32_t r0 = blockIdx.x * GM_TILE, ld = g.w.ld, xld = g.x_ld ? g.x_ld : ld;
+    const T *w = (const T *)g.w.w + (size_t)row_base * ld, *x = (const T *)g.x + (g.block_rows ? (size_t)(r0 / g.block_rows) * ld : 0);
     const uint32_t tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
     float acc[4][4] = {};
     for (uint32_t k0 = 0; k0 < ld; k0 += GM_K) {
         for (uint32_t i = threadIdx.x; i < GM_TILE * GM_K; i += 256) {
             const uint32_t r = i / GM_K, k = i % GM_K;
             ws[k][r] = r0 + r < rows ? Elem<T>::to(w[(size_t)(r0 + r) * ld + k0 + k]) : 0.0f;
-            xs[k][r] = first + r < end ? Elem<T>::to(x[(size_t)(first + r) * ld + k0 + k]) : 0.0f;
+            xs[k][r] = first + r < end ? Elem<T>::to(x[(size_t)(first + r) * xld + k0 + k]) : 0.0f;
         }
         __syncthreads();
 #pragma unroll
@@ -61,7 +61,7 @@ __global__ void __launch_bounds__(256) dense_gemm_kernel(DenseGemm g) {
     }
 }
 
-// The experts' gated unit over gathered columns: pre [n][2 ff_p] -> out [n][ff_p].
+// The gated unit over columns: pre [n][2 ff_p] -> out [n][ff_p].
 template <class T>
 __global__ void __launch_bounds__(256) gated_unit_kernel(const float *pre, uint32_t n, uint32_t ff_p, const float *col_scale, ExpertAct a, T *out) {
     pdl_trigger();
@@ -82,7 +82,7 @@ int32_t launch_dense_gemm(const DenseGemm &g, cudaStream_t st) {
     if (taken) return CERA_CUDA_OK;
     if (g.out_kind == DENSE_GATED_UNIT) {
         // the products into a stream-ordered scratch, then the unit
-        const uint32_t ff_p = g.rows_per_expert / 2;
+        const uint32_t ff_p = (g.tiles ? g.rows_per_expert : g.w.rows) / 2;
         float *pre = nullptr;
         CERA_CUDA_TRY(cudaMallocAsync((void **)&pre, (size_t)g.n * 2 * ff_p * 4, st));
         DenseGemm p = g;

@@ -5,7 +5,7 @@
 // MMAs run into the other accumulator.
 //
 // Grouped by expert the tiles come from a device-built work list.  With NA = 2 a stage holds two weight tiles (an expert's
-// gate rows and the same up rows) against one activation tile, and the epilogue forms the gated unit from the two
+// gate rows and the same up rows; without groups, the matrix's first and second half) against one activation tile, and the epilogue forms the gated unit from the two
 // accumulators.  Every wait is bounded (tma.cuh); a wait that runs out empties the CTA and raises a status bit.
 #include <cudaTypedefs.h>
 
@@ -17,7 +17,7 @@ namespace cera {
 
 __device__ unsigned int g_dense_tc_status = 0;
 
-// bits 17..19: roles of this kernel (loader, MMA, epilogue); bits 20..22: the prompt attention's (latent_prefill.cu)
+// bits 17..19: roles of this kernel (loader, MMA, epilogue); bits 20..22: the prompt attention's (attention_tc.cu)
 static const bool g_dense_tc_registered = register_kernel_status([] {
     unsigned int v = 0;
     cudaMemcpyFromSymbol(&v, g_dense_tc_status, sizeof(v));
@@ -76,7 +76,7 @@ __device__ __forceinline__ DtTile dt_tile(const DtParams &p, uint32_t t) {
         o.end = m.first + m.count;
     } else {
         o.row0 = o.a_row = (t / p.col_tiles) * DT_BM;
-        o.rows = p.g.w.rows;
+        o.rows = p.g.w.rows / NA;
         o.first = (t % p.col_tiles) * BN;
         o.end = min(o.first + BN, p.g.n);
     }
@@ -121,6 +121,7 @@ __global__ void __launch_bounds__(DT_THREADS, 1) dense_gemm_tc_kernel(const __gr
             bool ok = true;
             for (uint32_t t = blockIdx.x; t < n_tiles && ok; t += gridDim.x) {
                 const DtTile o = dt_tile<BN, NA>(p, t);
+                const uint32_t x0 = p.g.block_rows ? o.a_row / p.g.block_rows * p.g.w.ld : 0;
                 for (uint32_t k = 0; k < n_k; ++k, ++it) {
                     const uint32_t s = it % S::STAGES;
                     if (!(ok = tma::mbar_wait_blocking(empty + s, (it / S::STAGES & 1) ^ 1, abort_flag, &g_dense_tc_status, 1u))) break;
@@ -128,7 +129,7 @@ __global__ void __launch_bounds__(DT_THREADS, 1) dense_gemm_tc_kernel(const __gr
                     tma::mbar_expect_tx(full + s, S::STAGE);
                     tma::tensor_g2s_2d(st, &map_w, k * DT_KS, o.a_row, full + s);
                     if (NA == 2) tma::tensor_g2s_2d(st + DT_A_BYTES, &map_w, k * DT_KS, o.a_row + o.rows, full + s);
-                    tma::tensor_g2s_2d(st + NA * DT_A_BYTES, &map_x, k * DT_KS, o.first, full + s);
+                    tma::tensor_g2s_2d(st + NA * DT_A_BYTES, &map_x, x0 + k * DT_KS, o.first, full + s);
                 }
             }
             // given up: this CTA's shared memory must outlive the copies in flight
@@ -233,10 +234,10 @@ int32_t launch_tc(const DenseGemm &g, cudaStream_t st) {
     using S = Tile<BN, NA>;
     CUtensorMap mw, mx;
     CERA_TRY(tensor_map_bf16(&mw, g.w.w, g.w.rows, g.w.ld, DT_KS, DT_BM));
-    CERA_TRY(tensor_map_bf16(&mx, g.x, g.n, g.w.ld, DT_KS, BN));
+    CERA_TRY(tensor_map_bf16(&mx, g.x, g.n, g.row_len(), DT_KS, BN));
     DtParams p;
     p.g = g;
-    const uint32_t rows = g.tiles ? g.rows_per_expert / NA : g.w.rows;
+    const uint32_t rows = (g.tiles ? g.rows_per_expert : g.w.rows) / NA;
     p.row_tiles = (rows + DT_BM - 1) / DT_BM;
     p.col_tiles = g.tiles ? g.max_tiles : (g.n + BN - 1) / BN;
     const uint64_t tiles = (uint64_t)p.row_tiles * p.col_tiles;
@@ -260,6 +261,7 @@ int32_t launch_dense_gemm_tc(const DenseGemm &g, cudaStream_t st, bool *taken) {
         if (g.group_columns <= 64) return pair ? launch_tc<64, 2>(g, st) : launch_tc<64, 1>(g, st);
         return pair ? launch_tc<128, 2>(g, st) : launch_tc<128, 1>(g, st);
     }
+    if (pair) return g.n <= 32 ? launch_tc<32, 2>(g, st) : g.n <= 64 ? launch_tc<64, 2>(g, st) : launch_tc<128, 2>(g, st);
     const uint32_t row_tiles = (g.w.rows + DT_BM - 1) / DT_BM;
     if (g.n <= 32) return launch_tc<32, 1>(g, st);
     if (g.n <= 64) return launch_tc<64, 1>(g, st);

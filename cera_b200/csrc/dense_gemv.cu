@@ -1,77 +1,13 @@
 // One-column products with dense weights: the decode step's projections, with the work that follows them fused where
-// one warp holds all a result needs (the minGRU update, the experts' gated unit, the sum over picks).
-//
-// A row group (R rows that share the activation vector) is walked by WPR warps of a CTA, 16 bytes per lane and row at a
-// time; the first loads are issued before the kernel waits for its predecessor (weights never change).
-#include "dense.cuh"
+// one warp holds all a result needs (the minGRU update, the gated units, the sum over picks).
+#include "dense_gemv.cuh"
 #include "moe_route.cuh"
 
 namespace cera {
 
 namespace {
 
-constexpr int GV_WARPS = 8;
-
-template <class T, int R, int U>
-struct RowDot {
-    const T *w[R];
-    uint32_t nv, step, c;
-    uint4 buf[R][U];
-    // part of `parts` warps that share the row; ld elements per row
-    __device__ __forceinline__ void start(uint32_t ld, int part, int parts) {
-        nv = ld / Elem<T>::N;
-        step = 32u * parts;
-        c = part * 32u + (threadIdx.x & 31);
-    }
-    __device__ __forceinline__ void fetch() {
-#pragma unroll
-        for (int u = 0; u < U; ++u)
-            if (c + u * step < nv) {
-#pragma unroll
-                for (int r = 0; r < R; ++r) buf[r][u] = ld_stream(reinterpret_cast<const uint4 *>(w[r]) + c + u * step);
-            }
-    }
-    __device__ __forceinline__ void run(const T *x, float (&acc)[R]) {
-        while (c < nv) {
-#pragma unroll
-            for (int u = 0; u < U; ++u)
-                if (c + u * step < nv) {
-                    float xf[Elem<T>::N], wf[Elem<T>::N];
-                    Elem<T>::unpack(*(reinterpret_cast<const uint4 *>(x) + c + u * step), xf);
-#pragma unroll
-                    for (int r = 0; r < R; ++r) {
-                        Elem<T>::unpack(buf[r][u], wf);
-#pragma unroll
-                        for (int i = 0; i < Elem<T>::N; ++i) acc[r] = fmaf(wf[i], xf[i], acc[r]);
-                    }
-                }
-            c += U * step;
-            fetch();
-        }
-    }
-};
-
-// Sums of R values over the WPR warps of a group; valid in lane 0 of the group's first warp.
-template <int R, int WPR>
-__device__ __forceinline__ void group_sum(float (&acc)[R], float (*red)[R]) {
-#pragma unroll
-    for (int r = 0; r < R; ++r) acc[r] = warp_sum(acc[r]);
-    if (WPR == 1) return;
-    const int warp = threadIdx.x >> 5;
-    if ((threadIdx.x & 31) == 0) {
-#pragma unroll
-        for (int r = 0; r < R; ++r) red[warp][r] = acc[r];
-    }
-    __syncthreads();
-    if (warp % WPR == 0) {
-#pragma unroll
-        for (int r = 0; r < R; ++r) {
-            acc[r] = 0.0f;
-#pragma unroll
-            for (int i = 0; i < WPR; ++i) acc[r] += red[warp + i][r];
-        }
-    }
-}
+using namespace gv;
 
 template <class T, int R, int WPR>
 __global__ void __launch_bounds__(GV_WARPS * 32) gemv_kernel(const T *__restrict__ w, uint32_t rows, uint32_t ld, const T *x, float *y) {
@@ -118,6 +54,25 @@ __global__ void __launch_bounds__(GV_WARPS * 32) mingru_step_kernel(const T *__r
         state[g] = s;
         out[g] = Elem<T>::from(s * silu_f32(acc[2]));
     }
+}
+
+// Rows [0, ff_p) gate, [ff_p, 2 ff_p) up of w; out = unit(gate, up).
+template <class T, int WPR>
+__global__ void __launch_bounds__(GV_WARPS * 32) gated_unit_step_kernel(const T *__restrict__ w, uint32_t ff_p, uint32_t ld, const T *x, ExpertAct a, T *out) {
+    __shared__ float red[GV_WARPS][2];
+    pdl_trigger();
+    const int warp = threadIdx.x >> 5;
+    const uint32_t g = blockIdx.x * (GV_WARPS / WPR) + warp / WPR, gi = min(g, ff_p - 1);
+    RowDot<T, 2, 4> d;
+    d.w[0] = w + (size_t)gi * ld;
+    d.w[1] = d.w[0] + (size_t)ff_p * ld;
+    d.start(ld, warp % WPR, WPR);
+    d.fetch();
+    pdl_wait();
+    float acc[2] = {};
+    d.run(x, acc);
+    group_sum<2, WPR>(acc, red);
+    if (warp % WPR == 0 && (threadIdx.x & 31) == 0 && g < ff_p) out[g] = Elem<T>::from(gated_unit(acc[0], acc[1], a));
 }
 
 // grid (row groups, picks).  Every CTA repeats the pick from the router logits; CTA 0 of a pick leaves it for the down step.
@@ -196,30 +151,6 @@ __global__ void __launch_bounds__(GV_WARPS * 32) expert_down_kernel(const T *__r
     if (warp % WPR == 0 && (threadIdx.x & 31) == 0 && g < rows) y[g] = total[0];
 }
 
-// Warps per row group: shared further while every warp keeps a batch of loads (u vectors a lane) and all groups still run
-// at once; few groups are shared whatever the batch.
-int pick_wpr(size_t groups, size_t row_bytes, int u) {
-    const size_t vecs = row_bytes / 16, few = (size_t)sm_count() * 14, room = (size_t)sm_count() * 64;
-    int wpr = 1;
-    while (wpr < 8 && (groups * wpr < few || (groups * wpr * 2 <= room && vecs >= (size_t)wpr * 2 * 32 * u))) wpr *= 2;
-    return wpr;
-}
-
-template <class F>
-int32_t with_wpr(int wpr, F f) {
-    switch (wpr) {
-        case 1: return f(std::integral_constant<int, 1>{});
-        case 2: return f(std::integral_constant<int, 2>{});
-        case 4: return f(std::integral_constant<int, 4>{});
-        default: return f(std::integral_constant<int, 8>{});
-    }
-}
-template <class F>
-int32_t with_type(int f32, F f) {
-    return f32 ? f(float{}) : f(bf16{});
-}
-dim3 gv_grid(size_t groups, int wpr, uint32_t y = 1) { return dim3((unsigned)((groups * wpr + GV_WARPS - 1) / GV_WARPS), y); }
-
 }  // namespace
 
 int32_t launch_dense_gemv(const DenseView &w, const void *x, float *y, cudaStream_t st) {
@@ -248,6 +179,20 @@ int32_t launch_mingru_step(const DenseView &w, const void *x, const float *z_bia
             return check_cuda(launch_k(mingru_step_kernel<T, decltype(n)::value>, gv_grid(wp, wpr), dim3(GV_WARPS * 32), 0, st, (const T *)w.w, wp, w.ld,
                                        (const T *)x, z_bias, x_bias, state, (T *)out),
                               "mingru step launch");
+        });
+    });
+}
+
+int32_t launch_gated_unit_step(const DenseView &w, const void *x, const ExpertAct &a, void *out, cudaStream_t st) {
+    const uint32_t ff_p = w.rows / 2;
+    const int wpr = pick_wpr(ff_p, (size_t)w.ld * (w.f32 ? 4 : 2), 4);
+    count_launch();
+    return with_type(w.f32, [&](auto t) {
+        using T = decltype(t);
+        return with_wpr(wpr, [&](auto n) {
+            return check_cuda(launch_k(gated_unit_step_kernel<T, decltype(n)::value>, gv_grid(ff_p, wpr), dim3(GV_WARPS * 32), 0, st, (const T *)w.w, ff_p,
+                                       w.ld, (const T *)x, a, (T *)out),
+                              "gated unit launch");
         });
     });
 }

@@ -561,12 +561,6 @@ int32_t latent_attention(const float *q32, const LatentShape &s, const void *uk,
 
 }  // namespace
 
-uint32_t latent_splits(size_t n_positions) {
-    uint32_t s = 1;
-    while (s < LATENT_MAX_SPLITS && s * LM_KEYS < n_positions) s *= 2;
-    return s;
-}
-
 int32_t launch_latent_prepare(const float *in, const LatentShape &s, size_t n, size_t start_pos, const uint32_t *pos_dev, const float *c_norm, float eps,
                               const float *rope_table, void *cache_c, void *cache_r, int f32, float *q32, void *qt, float *gate, cudaStream_t st) {
     if (n == 0) return CERA_CUDA_OK;
