@@ -34,12 +34,16 @@ class LayerDesc(C.Structure):
     _fields_ = [("mixer", _i32), ("ff", _i32), ("n_heads", _u32), ("head_dim", _u32), ("rot_dim", _u32), ("value_dim", _u32),
                 ("kv_rank", _u32), ("rope_base", _f), ("attn_scale", _f), ("recurrent_width", _u32), ("ff_width", _u32),
                 ("n_experts", _u32), ("n_used", _u32), ("act_limit", _f), ("act_alpha", _f), ("act_shift", _f),
-                ("router_softmax", _i32), ("router_renorm", _i32), ("weight_input", _i32)]
+                ("router_softmax", _i32), ("router_renorm", _i32), ("weight_input", _i32), ("n_kv_heads", _u32), ("softcap", _f),
+                ("qk_norm", _i32), ("attn_bias", _i32), ("n_blocks", _u32), ("conv_taps", _u32), ("decay", _f), ("state_size", _u32),
+                ("n_groups", _u32), ("n_norm_groups", _u32)]
 
 
 class LayeredConfig(C.Structure):
     _fields_ = [("n_layers", _u32), ("hidden_size", _u32), ("vocab_size", _u32), ("max_seq_len", _u32), ("norm_eps", _f),
-                ("dtype", _i32), ("device", _i32), ("bigram_buckets", _u32), ("bigram_mul_prev", _u64), ("bigram_mul_cur", _u64)]
+                ("dtype", _i32), ("device", _i32), ("bigram_buckets", _u32), ("bigram_mul_prev", _u64), ("bigram_mul_cur", _u64),
+                ("embedding_scale", _f), ("norm_offset", _f), ("tied_output", _i32), ("no_post_norms", _i32), ("loop_start", _u32),
+                ("loop_stop", _u32), ("loop_times", _u32)]
 
 
 # name -> (restype, argtypes); every symbol include/cera_cuda.h declares.

@@ -9,7 +9,6 @@ import os
 
 from .layered import LayerDesc, LayeredModel, Mixer, Ff
 from .model import Role
-from .safetensors import SafetensorsFile
 
 # the expert unit: min(g) * sigmoid(ALPHA g) * (u + SHIFT)
 ACT_ALPHA = 1.702
@@ -79,10 +78,5 @@ def load_goletar(path, config=None, max_seq_len=4096, dtype="bfloat16", device=0
             config = json.load(f)
     kw, layers = describe(config)
     model = LayeredModel(layers, max_seq_len=max_seq_len, dtype=dtype, device=device, **kw)
-    with SafetensorsFile(os.path.join(path, "model.safetensors")) as f:
-        for name, role, layer, expert in tensor_roles(layers):
-            rows, cols, kind, data = f.get(name)
-            model.add_tensor(role, layer, kind, rows, cols, data, expert=expert)
-            del data
-    model.finalize()
+    model.load(path, tensor_roles(layers))
     return model

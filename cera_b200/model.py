@@ -45,6 +45,25 @@ class Role(enum.IntEnum):
     EXPERT_GATE = 41
     EXPERT_UP = 42
     EXPERT_DOWN = 43
+    ATTN_Q_BIAS = 50
+    ATTN_K_BIAS = 51
+    ATTN_V_BIAS = 52
+    CONV = 54
+    CONV_BIAS = 55
+    LRU_OUT = 60
+    LRU_OUT_BIAS = 61
+    LRU_IN = 62
+    LRU_IN_BIAS = 63
+    LRU_DECAY_GATE = 64
+    LRU_DECAY_GATE_BIAS = 65
+    LRU_INPUT_GATE = 66
+    LRU_INPUT_GATE_BIAS = 67
+    LRU_LAMBDA = 68
+    SSM_IN = 70
+    SSM_DT_BIAS = 71
+    SSM_A_LOG = 72
+    SSM_D = 73
+    SSM_NORM = 74
 
 
 ModelConfig = Config

@@ -10,13 +10,18 @@ def _goletar(path, config, **kw):
     return load_goletar(path, config, **kw)
 
 
+def _piditar(path, config, **kw):
+    from .piditar import load_piditar
+    return load_piditar(path, config, **kw)
+
+
 def _llama(path, _config, dtype=None, **kw):
     if dtype not in (None, "quantized"):
         raise ValueError(f"a GGUF model runs its own quantized weights, not {dtype}")
     return load_llama(path, **kw)
 
 
-FOLDER_ARCHITECTURES = {"Goletar": _goletar}
+FOLDER_ARCHITECTURES = {"Goletar": _goletar, "Piditar": _piditar}
 GGUF_ARCHITECTURES = {a: _llama for a in ("llama", "qwen2", "qwen3", "granite")}
 
 

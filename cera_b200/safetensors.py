@@ -1,5 +1,6 @@
 """Safetensors reader: the file is mapped and tensors are handed out as raw views, as gguf.py does for GGUF."""
 import json
+import math
 import mmap
 import struct
 
@@ -51,12 +52,13 @@ class SafetensorsFile:
         return self.tensors[name][0]
 
     def get(self, name):
-        """(rows, cols, ggml type, raw bytes): vectors are one row, scalars one number."""
+        """(rows, cols, ggml type, raw bytes): vectors are one row, scalars one number, stacked matrices one tall matrix."""
         shape = self.shape(name)
         _, kind, off, nbytes = self.tensors[name]
-        if len(shape) > 2 or kind is None:
-            raise SafetensorsError(f"tensor {name} of shape {shape} is not a float vector or matrix")
-        rows, cols = (1, 1) if not shape else (1, shape[0]) if len(shape) == 1 else shape
+        if kind is None:
+            raise SafetensorsError(f"tensor {name} is an integer table")
+        cols = shape[-1] if shape else 1
+        rows = math.prod(shape[:-1])
         return rows, cols, kind, np.frombuffer(self._buf, dtype=np.uint8, count=nbytes, offset=off)
 
     def close(self):

@@ -281,13 +281,33 @@ enum {
     CERA_ROLE_ROUTER = 40,         /* [experts][hidden] */
     CERA_ROLE_EXPERT_GATE = 41,    /* one expert's [ff_width][hidden] (cera_cuda_model_add_expert_tensor) */
     CERA_ROLE_EXPERT_UP = 42,
-    CERA_ROLE_EXPERT_DOWN = 43     /* [hidden][ff_width] */
+    CERA_ROLE_EXPERT_DOWN = 43,    /* [hidden][ff_width] */
+    /* grouped attention: ATTN_Q, ATTN_K, ATTN_V above and their biases; a layer's one gated unit: FFN_GATE, FFN_UP, FFN_DOWN */
+    CERA_ROLE_ATTN_Q_BIAS = 50,    /* [heads * head_dim] */
+    CERA_ROLE_ATTN_K_BIAS = 51,
+    CERA_ROLE_ATTN_V_BIAS = 52,
+    CERA_ROLE_CONV = 54,           /* [channels][taps], the last tap meets the current position */
+    CERA_ROLE_CONV_BIAS = 55,
+    CERA_ROLE_LRU_OUT = 60,        /* [recurrent_width][hidden]: the branch that gates the output */
+    CERA_ROLE_LRU_OUT_BIAS = 61,
+    CERA_ROLE_LRU_IN = 62,         /* [recurrent_width][hidden]: the convolved branch */
+    CERA_ROLE_LRU_IN_BIAS = 63,
+    CERA_ROLE_LRU_DECAY_GATE = 64, /* [blocks * block][block], block = recurrent_width / n_blocks */
+    CERA_ROLE_LRU_DECAY_GATE_BIAS = 65,
+    CERA_ROLE_LRU_INPUT_GATE = 66,
+    CERA_ROLE_LRU_INPUT_GATE_BIAS = 67,
+    CERA_ROLE_LRU_LAMBDA = 68,     /* [recurrent_width] */
+    CERA_ROLE_SSM_IN = 70,         /* rows z | x | B | C | step sizes */
+    CERA_ROLE_SSM_DT_BIAS = 71,    /* [heads] */
+    CERA_ROLE_SSM_A_LOG = 72,
+    CERA_ROLE_SSM_D = 73,
+    CERA_ROLE_SSM_NORM = 74        /* [heads * value_dim] */
 };
 
 /* A decoder described layer by layer: each layer names its token mixer and its feed-forward with their sizes and
  * constants.  Weights are dense (bf16 or f32).  No counterpart in the reference. */
-enum { CERA_MIXER_LATENT_ATTENTION = 1, CERA_MIXER_MINGRU = 2 };
-enum { CERA_FF_NONE = 0, CERA_FF_MOE = 1 };
+enum { CERA_MIXER_LATENT_ATTENTION = 1, CERA_MIXER_MINGRU = 2, CERA_MIXER_ATTENTION = 3, CERA_MIXER_RGLRU = 4, CERA_MIXER_SSM = 5 };
+enum { CERA_FF_NONE = 0, CERA_FF_MOE = 1, CERA_FF_GATED = 2 };
 typedef struct {
     int32_t mixer;
     int32_t ff;
@@ -306,6 +326,20 @@ typedef struct {
     uint32_t ff_width, n_experts, n_used;
     float act_limit, act_alpha, act_shift;
     int32_t router_softmax, router_renorm, weight_input;
+    /* CERA_FF_GATED: one such unit of width ff_width (act_limit inf, act_alpha 1, act_shift 0: silu(gate) * up).
+     * Grouped attention: n_heads query heads of head_dim / value_dim share n_kv_heads keys and values; the first rot_dim
+     * dimensions of q and k rotate as above; qk_norm: q and k are then divided by their root mean square per head;
+     * score = q k attn_scale, with softcap != 0 softcap * tanh(score / softcap). */
+    uint32_t n_kv_heads;
+    float softcap;
+    int32_t qk_norm, attn_bias;
+    /* real-gated linear recurrence: recurrent_width channels in n_blocks gate blocks, a causal convolution of conv_taps ahead;
+     * S = a S + sqrt(1 - a^2) i u, log a = -decay * r * softplus(lambda), result S * gelu(y) (tanh form) */
+    uint32_t n_blocks, conv_taps;
+    float decay;
+    /* state-space recurrence: n_heads heads of value_dim, state_size rows of state, B and C shared by n_heads / n_groups heads,
+     * conv_taps ahead; the gated result is normed in n_norm_groups parts */
+    uint32_t state_size, n_groups, n_norm_groups;
 } cera_cuda_layer_desc;
 
 typedef struct {
@@ -317,6 +351,13 @@ typedef struct {
      * buckets == 0: none */
     uint32_t bigram_buckets;
     uint64_t bigram_mul_prev, bigram_mul_cur;
+    float embedding_scale;   /* multiplies the token row; 0: 1 */
+    float norm_offset;       /* added to the stored weight of the sublayer norms and the final norm */
+    int32_t tied_output;     /* the head is the embedding table (without its scale) */
+    int32_t no_post_norms;   /* sublayers are normed before only */
+    /* layers [loop_start, loop_stop) run loop_times times in a row, each pass with a state of its own; before every pass but
+     * the first the embedding is added to the residual.  loop_times <= 1: once */
+    uint32_t loop_start, loop_stop, loop_times;
 } cera_cuda_layered_config;
 
 CERA_API int32_t cera_cuda_model_create(const cera_cuda_config *cfg, cera_cuda_model **out);
