@@ -413,21 +413,23 @@ def roofline_traffic():
         return {"bytes": None, "source": "profiles/roofline_traffic.json missing"}
 
 
-GOLETAR_SIZES = {"2048": dict(width=2048, n_layers=8), "4096": dict(width=4096, n_layers=8)}
+LAYERED_SIZES = {"2048": dict(width=2048, n_layers=8), "4096": dict(width=4096, n_layers=8)}
 
 
-def goletar_bench(which, size, n_layers, prompts, contexts, steps):
-    """Prompt and decode throughput of a Goletar model (bf16, random weights, layers of real-model shapes) or, which == "llama",
-    of the closest dense model at equal width, depth, vocabulary and active feed-forward width (Q4_K / Q6_K).  Prompts: one warm
+def layered_bench(which, size, n_layers, prompts, contexts, steps):
+    """Prompt and decode throughput of a Goletar or Piditar model (bf16, random weights, layers of real-model shapes) or, which ==
+    "llama", of the dense model, all at equal width, depth, vocabulary and active feed-forward width (dense: Q4_K / Q6_K).  Prompts: one warm
     pass, then the best of three through forward_prefill, host clock around the synchronous call.  Decode: chained greedy steps, CUDA events."""
     import torch
     from cera_b200 import synth
-    s = dict(GOLETAR_SIZES[size])
+    s = dict(LAYERED_SIZES[size])
     s["n_layers"] = n_layers or s["n_layers"]
     cfg = synth.goletar_config(**s)
     max_seq = max(prompts + [c + 2 * steps + 8 for c in contexts]) + 8
     if which == "goletar":
         model = synth.build_goletar(cfg, max_seq_len=max_seq)
+    elif which == "piditar":
+        model = synth.build_piditar(synth.piditar_config(**s), max_seq_len=max_seq)
     else:
         mlp = cfg["layers"][0]["mlp"]
         w = s["width"]
@@ -657,10 +659,10 @@ def main():
     ap.add_argument("--no-alt", action="store_true", help="skip the leg that re-runs the benchmark on the toleranced decode kernels")
     ap.add_argument("--no-stream-check", action="store_true", help="report a stream that differs from the reference's instead of failing")
     ap.add_argument("--gemm-case", default=None, help="with --only gemm-sweep: a single case type:m:k:n:image (e.g. q4_k:14336:4096:512:1)")
-    ap.add_argument("--only", default=None, choices=["roofline", "gemv-sweep", "gemm-sweep", "moe", "attn-sweep", "prefill", "goletar"],
+    ap.add_argument("--only", default=None, choices=["roofline", "gemv-sweep", "gemm-sweep", "moe", "attn-sweep", "prefill", "goletar", "piditar"],
                     help="run just the dominant-kernel microbench (the case ncu captures are taken on)")
-    ap.add_argument("--goletar-case", default=None,
-                    help="with --only goletar: a single case model:width:layers:prompt:context:steps (prompt or context 0: left out), e.g. llama:4096:2:512:0:0")
+    ap.add_argument("--layered-case", default=None,
+                    help="with --only goletar or piditar: a single case model:width:layers:prompt:context:steps (prompt or context 0: left out), e.g. llama:4096:2:512:0:0")
     ap.add_argument("--iters", type=int, default=200, help="timed launches of the kernel microbench")
     args = ap.parse_args()
     rank = int(os.environ.get("RANK", 0))
@@ -726,16 +728,16 @@ def main():
         dt = time.perf_counter() - t0
         emit(json.dumps({"prompt_len": args.prompt_len, "batched_prefill_s": round(dt, 4), "tok_s": round(args.prompt_len / dt, 1)}))
         model.close()
-    elif args.only == "goletar":
-        if args.goletar_case:
-            which, size, layers, prompt, ctx, steps = args.goletar_case.split(":")
-            emit(json.dumps(goletar_bench(which, size, int(layers), [int(prompt)] if int(prompt) else [], [int(ctx)] if int(ctx) else [], int(steps))))
+    elif args.only in ("goletar", "piditar"):
+        if args.layered_case:
+            which, size, layers, prompt, ctx, steps = args.layered_case.split(":")
+            emit(json.dumps(layered_bench(which, size, int(layers), [int(prompt)] if int(prompt) else [], [int(ctx)] if int(ctx) else [], int(steps))))
         else:
             sampler = ClockSampler(0)
             sampler.start()
-            for size in GOLETAR_SIZES:
-                for which in ("goletar", "llama"):
-                    emit(json.dumps(goletar_bench(which, size, None, [128, 512, 2048], [512, 4096], 64)))
+            for size in LAYERED_SIZES:
+                for which in ("goletar", "llama") if args.only == "goletar" else ("piditar", "goletar", "llama"):
+                    emit(json.dumps(layered_bench(which, size, None, [128, 512, 2048], [512, 4096], 64)))
             emit(json.dumps({"clocks": sampler.stop()}))
     elif args.only == "moe":
         import torch

@@ -19,15 +19,15 @@ __device__ __forceinline__ float gelu_tanh_f32(float x) {
     // 0.5 (1 + tanh z) = sigmoid(2 z)
     return x * sigmoid_f32(2.0f * 0.79788456080286535588f * (x + 0.044715f * x * x * x));
 }
-// a and the input term's factor from the raw gates; sp = decay * softplus(lam)
-__device__ __forceinline__ void rglru_gates(float r_raw, float i_raw, float sp, float &a, float &gain) {
-    const float m = sp * sigmoid_f32(r_raw);  // -log a
-    a = expf(-m);
-    // 1 - a^2 = 1 - e^-q: its Taylor series where the difference would cancel
-    const float q = 2.0f * m;
-    const float series = q * (1.0f - q * (1.0f / 2) * (1.0f - q * (1.0f / 3) * (1.0f - q * (1.0f / 4) * (1.0f - q * (1.0f / 5) * (1.0f - q * (1.0f / 6))))));
-    gain = sqrtf(q < 0.125f ? series : 1.0f - a * a) * sigmoid_f32(i_raw);
+// log a, a - 1 and the input term's factor from the raw gates; sp = decay * softplus(lam).  Slow channels have a within a few
+// units of rounding of 1: a - 1 keeps what a itself would lose, step after step.
+__device__ __forceinline__ void rglru_gates(float r_raw, float i_raw, float sp, float &log_a, float &am1, float &gain) {
+    log_a = -sp * sigmoid_f32(r_raw);
+    am1 = expm1f(log_a);
+    gain = sqrtf(-am1 * (2.0f + am1)) * sigmoid_f32(i_raw);  // 1 - a^2 = (1 - a)(1 + a)
 }
+// a s + input
+__device__ __forceinline__ float decayed(float am1, float s, float input) { return s + fmaf(am1, s, input); }
 
 // grid (groups of 8 channels of a block, blocks)
 template <class T>
@@ -56,9 +56,9 @@ __global__ void __launch_bounds__(GV_WARPS * 32) rglru_step_kernel(const float *
     d.run(us, acc);
     group_sum<2, 1>(acc, nullptr);
     if (lane == 0) {
-        float a, gain;
-        rglru_gates(acc[0] + v.gate_bias[(size_t)b * 2 * bp + c], acc[1] + v.gate_bias[(size_t)b * 2 * bp + bp + c], sp, a, gain);
-        const float s = a * v.state[ch] + gain * Elem<T>::to(us[c]);
+        float log_a, am1, gain;
+        rglru_gates(acc[0] + v.gate_bias[(size_t)b * 2 * bp + c], acc[1] + v.gate_bias[(size_t)b * 2 * bp + bp + c], sp, log_a, am1, gain);
+        const float s = decayed(am1, v.state[ch], gain * Elem<T>::to(us[c]));
         v.state[ch] = s;
         out[ch] = Elem<T>::from(s * gelu_tanh_f32(pre[ch] + v.in_bias[ch]));
     }
@@ -90,23 +90,23 @@ __global__ void __launch_bounds__(RG_WARPS * 32) rglru_scan_kernel(const float *
             step(t, r, i, x);
         }
     };
-    float A = 1.0f, B = 0.0f;
+    float A = 0.0f, B = 0.0f;  // a segment: s -> e^A s + B
     walk([&](uint32_t t, const float *r, const float *i, const float *x) {
 #pragma unroll
         for (int k = 0; k < RG_U; ++k)
             if (t + k < t1) {
-                float a, gain;
-                rglru_gates(r[k] + br, i[k] + bi, sp, a, gain);
-                A *= a;
-                B = a * B + gain * x[k];
+                float log_a, am1, gain;
+                rglru_gates(r[k] + br, i[k] + bi, sp, log_a, am1, gain);
+                A += log_a;
+                B = decayed(am1, B, gain * x[k]);
             }
     });
-    sa[warp][lane] = A;
+    sa[warp][lane] = expm1f(A);
     sb[warp][lane] = B;
     const float s0 = v.state[c];
     __syncthreads();
     float s = s0;
-    for (uint32_t w = 0; w < warp; ++w) s = sa[w][lane] * s + sb[w][lane];
+    for (uint32_t w = 0; w < warp; ++w) s = decayed(sa[w][lane], s, sb[w][lane]);
     walk([&](uint32_t t, const float *r, const float *i, const float *x) {
         float y[RG_U];
 #pragma unroll
@@ -114,9 +114,9 @@ __global__ void __launch_bounds__(RG_WARPS * 32) rglru_scan_kernel(const float *
 #pragma unroll
         for (int k = 0; k < RG_U; ++k)
             if (t + k < t1) {
-                float a, gain;
-                rglru_gates(r[k] + br, i[k] + bi, sp, a, gain);
-                s = a * s + gain * x[k];
+                float log_a, am1, gain;
+                rglru_gates(r[k] + br, i[k] + bi, sp, log_a, am1, gain);
+                s = decayed(am1, s, gain * x[k]);
                 out[(size_t)(t + k) * wp + c] = Elem<T>::from(s * gelu_tanh_f32(y[k] + by));
             }
     });

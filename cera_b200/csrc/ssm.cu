@@ -1,6 +1,7 @@
 // State-space recurrence with a matrix state per head (Mamba-2): S = exp(-exp(A_log) dt) S + dt B x^T, y = S^T C + D x,
 // dt = softplus(raw + bias); x, B, C come convolved through silu, B and C are shared by the heads of a group.  This file: the
-// decode step, the token-by-token scan and the gated norm behind both.  States, step sizes and decays are f32.
+// decode step, the token-by-token scan and the gated norm behind both.  States, step sizes and decays are f32; a decay
+// next to 1 enters as its difference from 1.
 #include "dense_gemv.cuh"
 #include "ssm.cuh"
 
@@ -43,7 +44,7 @@ __global__ void __launch_bounds__(SS_WARPS * 32) ssm_step_kernel(const float *pr
         else bc[i] = val;
         if (is_x || keep_bc) ring[ch] = now;
     }
-    const float dt = softplus_f32(pre[s.off_dt() + h] + dt_bias), a = expf(-expf(a_log) * dt);
+    const float dt = softplus_f32(pre[s.off_dt() + h] + dt_bias), am1 = expm1f(-expf(a_log) * dt);
     __syncthreads();
     const float x = live ? xs[lane] : 0.0f, dx = dt * x;
     float acc = 0.0f;
@@ -59,7 +60,7 @@ __global__ void __launch_bounds__(SS_WARPS * 32) ssm_step_kernel(const float *pr
         for (int k = 0; k < U; ++k) {
             const uint32_t r = r0 + warp + k * SS_WARPS;
             if (r < N && live) {
-                const float now = fmaf(a, old[k], bc[r] * dx);
+                const float now = old[k] + fmaf(am1, old[k], bc[r] * dx);
                 S[(size_t)r * s.dim_p] = now;
                 acc = fmaf(now, bc[N + r], acc);
             }
@@ -103,15 +104,15 @@ __global__ void __launch_bounds__(SS_WARPS * 32) ssm_scan_kernel(const float *pr
             if (lane == 0) {
                 const float dt = softplus_f32(pre[(size_t)(t0 + t) * s.in_p + s.off_dt() + h] + dt_bias);
                 dts[t] = dt;
-                as[t] = expf(-expf(a_log) * dt);
+                as[t] = expm1f(-expf(a_log) * dt);
             }
         }
         __syncthreads();
         for (uint32_t t = 0; t < m; ++t) {
-            const float a = as[t], dx = dts[t] * xs[t][lane];
+            const float am1 = as[t], dx = dts[t] * xs[t][lane];
             float acc = 0.0f;
             for (uint32_t r = warp; r < N; r += SS_WARPS) {
-                const float now = fmaf(a, st[r * 32 + lane], bs[t * N + r] * dx);
+                const float old = st[r * 32 + lane], now = old + fmaf(am1, old, bs[t * N + r] * dx);
                 st[r * 32 + lane] = now;
                 acc = fmaf(now, cs[t * N + r], acc);
             }

@@ -116,6 +116,56 @@ def build_goletar(config, seed=0, dtype="bfloat16", **model_kw):
     return m
 
 
+def piditar_config(width, n_layers, vocab=32768, ff=None):
+    """A Piditar configuration whose layers have the shapes of a real model of this width: real-gated recurrence, attention with
+    heads of 128 in groups of four, real-gated recurrence, state-space recurrence with heads of 64 and a state of 128, in turn."""
+    mlp = {"kind": "dense", "ff": ff or 2 * width}
+    lru = {"type": "rglru", "mixer": {"width": width, "blocks": width // 256, "conv": 4}, "mlp": mlp}
+    att = {"type": "attention", "mlp": mlp,
+           "mixer": {"heads": width // 128, "kv_heads": width // 512, "dim": 128, "vdim": 128, "scale": 128.0 ** -0.5, "softcap": 50.0,
+                     "rot": {"base": 500000.0, "dims": 128}}}
+    ssm = {"type": "mamba2", "mixer": {"heads": width // 32, "vdim": 64, "state": 128, "groups": 8, "norm_groups": 8, "conv": 4}, "mlp": mlp}
+    return {"architecture": "Piditar", "width": width, "vocab": vocab, "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0},
+            "layers": [(lru, att, lru, ssm)[i % 4] for i in range(n_layers)], "loop": {"start": 0, "stop": 1, "times": 1}}
+
+
+def build_piditar(config, seed=0, dtype="bfloat16", **model_kw):
+    """A finalized Piditar model with random weights made on the device."""
+    from . import piditar
+    from .layered import LayeredModel, Mixer
+    from .types import BF16
+    kw, layers = piditar.describe(config)
+    m = LayeredModel(layers, dtype=dtype, **kw, **model_kw)
+    gen = torch.Generator(device="cuda").manual_seed(seed)
+    W = kw["hidden_size"]
+
+    def shape(role, d):
+        H, inner = d.n_heads, d.n_heads * d.value_dim
+        w, b = d.recurrent_width, d.recurrent_width // d.n_blocks if d.n_blocks else 0
+        channels = inner + 2 * d.n_groups * d.state_size if d.mixer == Mixer.SSM else w
+        return {Role.TOKEN_EMBD: (kw["vocab_size"], W), Role.OUTPUT_NORM: (1, W), Role.MIX_PRE_NORM: (1, W), Role.FF_PRE_NORM: (1, W),
+                Role.MIX_OUTPUT: (W, w if d.mixer == Mixer.RGLRU else inner), Role.FFN_GATE: (d.ff_width, W), Role.FFN_UP: (d.ff_width, W),
+                Role.FFN_DOWN: (W, d.ff_width), Role.ATTN_Q: (H * d.head_dim, W), Role.ATTN_K: (d.n_kv_heads * d.head_dim, W),
+                Role.ATTN_V: (d.n_kv_heads * d.value_dim, W), Role.ATTN_Q_BIAS: (1, H * d.head_dim), Role.ATTN_K_BIAS: (1, d.n_kv_heads * d.head_dim),
+                Role.ATTN_V_BIAS: (1, d.n_kv_heads * d.value_dim), Role.CONV: (channels, d.conv_taps), Role.CONV_BIAS: (1, channels),
+                Role.LRU_OUT: (w, W), Role.LRU_IN: (w, W), Role.LRU_OUT_BIAS: (1, w), Role.LRU_IN_BIAS: (1, w), Role.LRU_DECAY_GATE: (w, b),
+                Role.LRU_INPUT_GATE: (w, b), Role.LRU_DECAY_GATE_BIAS: (1, w), Role.LRU_INPUT_GATE_BIAS: (1, w), Role.LRU_LAMBDA: (1, w),
+                Role.SSM_IN: (inner + channels + H, W), Role.SSM_DT_BIAS: (1, H), Role.SSM_A_LOG: (1, H), Role.SSM_D: (1, H),
+                Role.SSM_NORM: (1, inner)}[role]
+
+    for _, role, layer, _ in piditar.tensor_roles(layers):
+        rows, cols = shape(role, layers[layer])
+        v = torch.randn(rows, cols, device="cuda", dtype=torch.bfloat16, generator=gen)
+        if rows > 1 and role != Role.TOKEN_EMBD:
+            v *= cols ** -0.5
+        elif role in (Role.OUTPUT_NORM, Role.MIX_PRE_NORM, Role.FF_PRE_NORM):
+            v.fill_(0.0)
+        m.add_tensor(role, layer, BF16, rows, cols, v)
+    torch.cuda.synchronize()
+    m.finalize()
+    return m
+
+
 def prompt_tokens(n, vocab, seed):
     """Uniform-random token ids, reproducible without numpy's generator state."""
     mask = (1 << 64) - 1

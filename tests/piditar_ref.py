@@ -158,3 +158,57 @@ def greedy(prompt, n, config, weights):
     for _ in range(n):
         toks.append(int(np.argmax(logits(toks, config, weights)[-1])))
     return toks[len(prompt):]
+
+
+# ---- random models ------------------------------------------------------------------------------------------------
+
+def tensor_shapes(config):
+    W = config["width"]
+    shapes = {"embed": (config["vocab"], W), "final.norm": (W,)}
+    for i, entry in enumerate(config["layers"]):
+        p, m = f"l{i}.", entry["mixer"]
+        shapes[p + "norm1"] = (W,)
+        if entry["type"] == "attention":
+            H, G, d, dv = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+            mix = {"q": (H * d, W), "q.b": (H * d,), "k": (G * d, W), "k.b": (G * d,), "v": (G * dv, W), "v.b": (G * dv,), "o": (W, H * dv)}
+        elif entry["type"] == "rglru":
+            n, B, c = m["width"], m["blocks"], m["conv"]
+            b = n // B
+            mix = {"y": (n, W), "y.b": (n,), "x": (n, W), "x.b": (n,), "conv": (n, c), "conv.b": (n,), "ra": (B, b, b), "ra.b": (B, b), "ri": (B, b, b),
+                   "ri.b": (B, b), "lam": (n,), "o": (W, n)}
+        else:
+            H, inner, gn = m["heads"], m["heads"] * m["vdim"], m["groups"] * m["state"]
+            mix = {"in": (2 * inner + 2 * gn + H, W), "conv": (inner + 2 * gn, m["conv"]), "conv.b": (inner + 2 * gn,), "dt_bias": (H,), "A_log": (H,),
+                   "D": (H,), "norm": (inner,), "o": (W, inner)}
+        shapes.update({p + "mix." + k: v for k, v in mix.items()})
+        if entry["mlp"] is not None:
+            ff = entry["mlp"]["ff"]
+            shapes.update({p + "norm2": (W,), p + "mlp.gate": (ff, W), p + "mlp.up": (ff, W), p + "mlp.down": (W, ff)})
+    return shapes
+
+
+def random_weights(config, seed):
+    """bf16-representable weights of a scale that keeps every branch alive, as float64."""
+    rng = np.random.default_rng(seed)
+    out = {}
+    for name, shape in tensor_shapes(config).items():
+        leaf, z = name.rsplit(".", 1)[-1], rng.standard_normal(shape)
+        if leaf in ("norm1", "norm2"):
+            v = 0.3 * z
+        elif leaf == "norm":
+            v = 0.3 * z + (0.0 if name == "final.norm" else 1.0)
+        elif leaf in ("embed", "lam", "D"):
+            v = z
+        elif leaf == "b":
+            v = 0.5 * z
+        elif leaf == "dt_bias":
+            v = z - 1.0
+        elif leaf == "A_log":
+            v = z - 1.0
+        elif leaf == "conv":
+            v = z / np.sqrt(shape[-1])
+        else:
+            gain = {"gate": 1.5, "up": 1.5, "in": 1.5, "x": 1.5, "y": 1.5}.get(leaf, 1.0)
+            v = gain * z / np.sqrt(shape[-1])
+        out[name] = from_bf16(to_bf16(np.asarray(v))).astype(F).reshape(shape)
+    return out
