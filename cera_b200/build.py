@@ -19,7 +19,8 @@ LIB = os.path.join(HERE, "libcera_cuda.so")
 # Everything that is not listed belongs to "quantized".
 PARTS = {"core": ["runtime.cu", "model.cu", "argmax.cu"],
          "layered": ["layered.cu", "dense.cu", "dense_gemv.cu", "dense_gemm.cu", "dense_gemm_tc.cu", "mingru.cu", "latent_attention.cu",
-                     "attention_tc.cu", "grouped_attention.cu", "conv.cu", "rglru.cu", "ssm.cu", "moe_route.cu"]}
+                     "attention_tc.cu", "grouped_attention.cu", "conv.cu", "rglru.cu", "ssm.cu", "ssm_chunk.cu",
+                     "moe_route.cu"]}
 ALL_PARTS = ("core", "layered", "quantized")
 # Translation units whose float arithmetic must not be contracted into FMAs.
 NO_FMAD = {"convert.cu"}

@@ -238,7 +238,7 @@ int32_t launch_rglru_step(const float *pre, const RglruView &v, const uint32_t *
 int32_t launch_rglru_scan(const float *pre, const void *u, const float *gate, const RglruView &v, size_t n, size_t start_pos, void *out, int f32,
                           cudaStream_t st);
 
-// ---- state-space recurrence with a matrix state per head (ssm.cu) ------------------------------------------------------------
+// ---- state-space recurrence with a matrix state per head (ssm.cu, ssm_chunk.cu) --------------------------------------------
 constexpr uint32_t SSM_MAX_STATE = 768;  // state_p at most (the scan's shared memory)
 struct SsmShape {
     uint32_t heads = 0, dim = 0, state = 0, groups = 0, norm_groups = 0;  // dim: values of a head
@@ -263,6 +263,9 @@ struct SsmView {
 int32_t launch_ssm_step(const float *pre, const SsmView &v, const uint32_t *pos_dev, float *y, int f32, cudaStream_t st);
 // A portion after launch_conv (xbc [n][channels] of T): y [n][inner_p].
 int32_t launch_ssm_scan(const float *pre, const void *xbc, const SsmView &v, size_t n, size_t start_pos, float *y, int f32, cudaStream_t st);
+// The same in chunks on the tensor cores (bf16).
+bool ssm_chunks_support(const SsmShape &s);
+int32_t launch_ssm_chunks(const float *pre, const void *xbc, const SsmView &v, size_t n, size_t start_pos, float *y, cudaStream_t st);
 // out = rms_norm of each of norm_groups parts of (y * silu(z)), times the weight; out [n][ldo] of T.
 int32_t launch_gated_norm(const float *y, const float *pre, const SsmView &v, size_t n, void *out, size_t ldo, int f32, cudaStream_t st);
 

@@ -1,7 +1,7 @@
 // Many-column bf16 products on the fifth-generation tensor cores: out[column][row] = W x, tcgen05.mma kind::f16 with f32
 // accumulators in TMEM.  A persistent CTA walks output tiles of 128 weight rows x BN columns (tokens): one thread keeps a
-// ring of stages filled by TMA (64 elements of k, 128-byte swizzle), one thread issues the MMAs, four warps drain the
-// finished accumulator - lane = weight row, so a column's 128 values leave as consecutive stores - while the next tile's
+// ring of stages filled by TMA (64 elements of k, 128-byte swizzle), one thread issues the MMAs, eight warps drain the
+// finished accumulator (two share its 32 rows and take turns at 32 columns) - lane = weight row, so a column's 128 values leave as consecutive stores - while the next tile's
 // MMAs run into the other accumulator.
 //
 // Grouped by expert the tiles come from a device-built work list.  With NA = 2 a stage holds two weight tiles (an expert's
@@ -43,7 +43,7 @@ int32_t tensor_map_bf16(CUtensorMap *map, const void *base, uint64_t rows, uint6
 
 namespace {
 
-constexpr int DT_BM = 128, DT_KS = 64, DT_THREADS = 6 * 32;  // loader, MMA, four epilogue warps
+constexpr int DT_BM = 128, DT_KS = 64, DT_THREADS = 10 * 32;  // loader, MMA, eight epilogue warps
 constexpr uint32_t DT_A_BYTES = DT_BM * DT_KS * 2;
 
 template <int BN, int NA>
@@ -100,7 +100,7 @@ __global__ void __launch_bounds__(DT_THREADS, 1) dense_gemm_tc_kernel(const __gr
         }
         for (int i = 0; i < 2; ++i) {
             tma::mbar_init(acc_full + i, 1);
-            tma::mbar_init(acc_empty + i, 4);
+            tma::mbar_init(acc_empty + i, 8);
         }
         *abort_flag = 0;
         tma::mbar_init_fence();
@@ -163,6 +163,7 @@ __global__ void __launch_bounds__(DT_THREADS, 1) dense_gemm_tc_kernel(const __gr
         }
     } else {
         const uint32_t quad = warp & 3;  // the TMEM lanes this warp may read: [32 quad, + 32)
+        const uint32_t turn = (warp - 2) >> 2;
         uint32_t j = 0;
         for (uint32_t t = blockIdx.x; t < n_tiles; t += gridDim.x, ++j) {
             const uint32_t b = j & 1;
@@ -173,7 +174,7 @@ __global__ void __launch_bounds__(DT_THREADS, 1) dense_gemm_tc_kernel(const __gr
             const uint32_t row = o.row0 + quad * 32 + lane, acc = tmem + b * S::ACC + (quad * 32 << 16), cols = o.end - o.first;
             const bool live = row < o.rows;
 #pragma unroll 1
-            for (uint32_t c0 = 0; c0 < BN && c0 < cols; c0 += 32) {
+            for (uint32_t c0 = turn * 32; c0 < BN && c0 < cols; c0 += 64) {
                 uint32_t v[2][16];
                 tmem_ld16(acc + c0, v[0]);
                 tmem_ld16(acc + c0 + 16, v[1]);

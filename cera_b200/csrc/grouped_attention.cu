@@ -221,11 +221,12 @@ __global__ void __launch_bounds__(GS_WARPS * 32) grouped_split_kernel(const floa
 
 // grid (heads, queries): the splits' sums under a common maximum.
 template <class T>
-__global__ void __launch_bounds__(128) grouped_merge_kernel(const float *part, GroupedShape s, uint32_t splits, T *out, size_t ldo) {
+__global__ void __launch_bounds__(256) grouped_merge_kernel(const float *part, GroupedShape s, uint32_t splits, T *out, size_t ldo) {
     __shared__ float wt[KV_MAX_SPLITS];
+    __shared__ float2 sums[8][32];
     pdl_trigger();
     pdl_wait();
-    const uint32_t h = blockIdx.x, j = blockIdx.y, lane = threadIdx.x & 31;
+    const uint32_t h = blockIdx.x, j = blockIdx.y, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const size_t ps = s.vdim_p + 2;
     const float *p = part + ((size_t)j * s.heads + h) * splits * ps;
     if (threadIdx.x < 32) {
@@ -251,11 +252,30 @@ __global__ void __launch_bounds__(128) grouped_merge_kernel(const float *part, G
             if (lane + 32 * i < splits) wt[lane + 32 * i] = ms[i] / den;
     }
     __syncthreads();
-    for (uint32_t d = threadIdx.x; d < s.vdim_p; d += 128) {
-        float acc = 0.0f;
+    for (uint32_t d0 = 0; d0 < s.vdim_p; d0 += 64) {  // a lane two values, a warp every eighth split
+        const uint32_t d = d0 + 2 * lane;
+        float2 acc = make_float2(0.0f, 0.0f);
+        if (d < s.vdim_p) {
 #pragma unroll 8
-        for (uint32_t i = 0; i < splits; ++i) acc = fmaf(wt[i], p[i * ps + 2 + d], acc);
-        out[j * ldo + (size_t)h * s.vdim_p + d] = Elem<T>::from(acc);
+            for (uint32_t i = warp; i < splits; i += 8) {
+                const float2 v = *reinterpret_cast<const float2 *>(p + i * ps + 2 + d);
+                acc.x = fmaf(wt[i], v.x, acc.x);
+                acc.y = fmaf(wt[i], v.y, acc.y);
+            }
+        }
+        sums[warp][lane] = acc;
+        __syncthreads();
+        if (warp == 0 && d < s.vdim_p) {
+#pragma unroll
+            for (int i = 1; i < 8; ++i) {
+                acc.x += sums[i][lane].x;
+                acc.y += sums[i][lane].y;
+            }
+            T *o = out + j * ldo + (size_t)h * s.vdim_p + d;
+            o[0] = Elem<T>::from(acc.x);
+            o[1] = Elem<T>::from(acc.y);
+        }
+        __syncthreads();
     }
 }
 
@@ -283,7 +303,7 @@ int32_t grouped_attention(const float *q32, const GroupedShape &s, const void *c
     };
     CERA_TRY(ni <= 1 ? go(grouped_split_kernel<T, 1>) : ni <= 2 ? go(grouped_split_kernel<T, 2>) : ni <= 4 ? go(grouped_split_kernel<T, 4>) : go(grouped_split_kernel<T, 8>));
     count_launch();
-    return check_cuda(launch_k(grouped_merge_kernel<T>, dim3(s.heads, (unsigned)n), dim3(128), 0, st, (const float *)part, s, splits, (T *)out, ldo), "attention merge launch");
+    return check_cuda(launch_k(grouped_merge_kernel<T>, dim3(s.heads, (unsigned)n), dim3(256), 0, st, (const float *)part, s, splits, (T *)out, ldo), "attention merge launch");
 }
 
 }  // namespace

@@ -7,6 +7,7 @@
 #include <type_traits>
 
 #include "dense.cuh"
+#include "mma.cuh"
 #include "tma.cuh"
 
 namespace cg = cooperative_groups;
@@ -239,18 +240,6 @@ __global__ void __launch_bounds__(LA_WARPS * 32) latent_split_kernel(const float
 // bf16 part (two products into one f32 accumulator).  Softmax in f32 over the CTA's tile; the weights enter the second
 // product as a high and a low part as well.  Weighted latents: warp = a quarter of the latent's columns, NP pairs of 8.
 constexpr int LM_KEYS = 64, LM_HEADS = 16, LM_P_LD = LM_KEYS + 8;
-
-__device__ __forceinline__ void ldsm4(uint32_t (&r)[4], const void *p) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(tma::smem_u32(p)) : "memory");
-}
-__device__ __forceinline__ void ldsm4_trans(uint32_t (&r)[4], const void *p) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(tma::smem_u32(p)) : "memory");
-}
-__device__ __forceinline__ void mma_bf16(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
 
 template <int NP>
 __global__ void __launch_bounds__(128) latent_split_mma_kernel(const bf16 *q, LatentShape s, const bf16 *cache_c, const bf16 *cache_r, uint32_t start_pos,

@@ -31,6 +31,8 @@ namespace {
 constexpr size_t LAYERED_CHUNK = 2048;   // prompt tokens per chunk
 constexpr size_t ATTENTION_TC_MIN = 16;  // shorter portions attend query by query
 
+constexpr size_t SSM_CHUNK_MIN = 16;      // shorter portions are scanned token by token
+
 struct ExpertFfn {
     DenseView gate_up, down, router;  // gate_up: per expert ff_p gate rows, ff_p up rows; router: f32
     uint32_t ff_p = 0;
@@ -825,7 +827,8 @@ int32_t LayeredModel::ssm_chunk(LayerRun &R, size_t n, size_t start_pos) {
     const SsmView v = ssm_view(R);
     const uint32_t channels = v.s.channels();
     CERA_TRY(launch_conv(pre + v.s.inner_p(), v.s.in_p, nullptr, v.conv, 1, n, start_pos, conv, channels, f32, stream));
-    CERA_TRY(launch_ssm_scan(pre, conv, v, n, start_pos, aux, f32, stream));
+    if (!f32 && n >= SSM_CHUNK_MIN && ssm_chunks_support(v.s)) CERA_TRY(launch_ssm_chunks(pre, conv, v, n, start_pos, aux, stream));
+    else CERA_TRY(launch_ssm_scan(pre, conv, v, n, start_pos, aux, f32, stream));
     return launch_gated_norm(aux, pre, v, n, mix, layers[R.layer].out.ld, f32, stream);
 }
 
