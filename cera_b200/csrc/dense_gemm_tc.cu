@@ -1,12 +1,12 @@
 // Many-column bf16 products on the fifth-generation tensor cores: out[column][row] = W x, tcgen05.mma kind::f16 with f32
 // accumulators in TMEM.  A persistent CTA walks output tiles of 128 weight rows x BN columns (tokens): one thread keeps a
 // ring of stages filled by TMA (64 elements of k, 128-byte swizzle), one thread issues the MMAs, eight warps drain the
-// finished accumulator (two share its 32 rows and take turns at 32 columns) - lane = weight row, so a column's 128 values leave as consecutive stores - while the next tile's
-// MMAs run into the other accumulator.
+// finished accumulator - lane = weight row, so a column's values leave as consecutive stores; two warps share 32 rows and
+// take 32 columns in turn - while the next tile's MMAs run into the other accumulator.
 //
 // Grouped by expert the tiles come from a device-built work list.  With NA = 2 a stage holds two weight tiles (an expert's
-// gate rows and the same up rows; without groups, the matrix's first and second half) against one activation tile, and the epilogue forms the gated unit from the two
-// accumulators.  Every wait is bounded (tma.cuh); a wait that runs out empties the CTA and raises a status bit.
+// gate rows and the same up rows; without groups, the matrix's first and second half) against one activation tile, and the
+// epilogue forms the gated unit from the two accumulators.  Every wait is bounded (tma.cuh); a wait that runs out empties the CTA and raises a status bit.
 #include <cudaTypedefs.h>
 
 #include "dense.cuh"

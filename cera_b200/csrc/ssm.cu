@@ -129,7 +129,7 @@ __global__ void __launch_bounds__(SS_WARPS * 32) ssm_scan_kernel(const float *pr
     }
     for (uint32_t r = warp; r < N; r += SS_WARPS)
         if (live) S[(size_t)r * s.dim_p] = st[r * 32 + lane];
-    ssm_keep(pre, v, h, p0, min(p0 + 32, s.dim_p), blockIdx.y == 0, n, start_pos);
+    ssm_keep(pre, v, h, p0, min(p0 + 32, s.dim_p), blockIdx.y == 0, n, start_pos, SS_WARPS * 32);
 }
 
 constexpr int GN_KEEP = 8;  // values a thread holds in registers

@@ -2,10 +2,12 @@
 // running sum of the log decays and S the state the chunk starts from,
 //   y_t = exp(L_t) S^T C_t + sum over j <= t of (C_t . B_j) exp(L_t - L_j) dt_j x_j + D x_t
 //   S  <- exp(L_end) S + sum over j of B_j (exp(L_end - L_j) dt_j x_j)^T
-// A CTA walks the chunks of one head (64 of its values); a warp owns 16 values for all tokens and all rows of the state, whose
-// f32 accumulators stay in registers from chunk to chunk and turn into operands of the first product as they are.  B, C and x
-// are bf16 as the convolution leaves them; decays, weights and states, f32, enter a product as a high and a low bf16 part.
-// L is summed in double and kept as two floats, so that close differences of large sums stay exact.
+// A CTA walks the chunks of one head (64 of its values).  Eight warps compute: a warp owns 16 values and half the rows of the
+// state, whose f32 accumulators stay in registers from chunk to chunk and turn into operands of the first product as they
+// are; the two halves of S^T C are exchanged through shared memory, each warp finishing two of the four 16-token tiles.  A
+// ninth warp works out the next chunk's decays meanwhile.  B, C and x are bf16 as the convolution leaves them; decays, weights
+// and states, f32, enter a product as a high and a low bf16 part.  L is summed in double and kept as two floats, so that
+// close differences of large sums stay exact.
 #include "mma.cuh"
 #include "ssm.cuh"
 
@@ -13,38 +15,81 @@ namespace cera {
 
 namespace {
 
-constexpr int SC_Q = 64, SC_P = 64, SC_WARPS = 4, SC_LD = SC_P + 8;
+constexpr int SC_Q = 64, SC_P = 64, SC_WARPS = 8, SC_LD = SC_P + 8;
 
 template <int NT>  // the state's rows / 16
 struct ChunkSmem {
     static constexpr int N = NT * 16, LD = N + 8;
     bf16 b[2][SC_Q][LD], c[2][SC_Q][LD], x[2][SC_Q][SC_LD];
     bf16 m[2][SC_Q][SC_LD], wx[2][SC_Q][SC_LD];  // high, low
-    float l_hi[SC_Q], l_lo[SC_Q], dt[SC_Q], w[SC_Q], e[SC_Q];
-    float e_end;
+    float4 half[SC_WARPS][4][32];  // of S^T C, for the warp that finishes the tile
+    float l_hi[2][SC_Q], l_lo[2][SC_Q], dt[2][SC_Q], w[2][SC_Q], e[2][SC_Q];
+    float e_end[2];
 };
 
 template <int NT>
-__global__ void __launch_bounds__(SC_WARPS * 32) ssm_chunk_kernel(const float *pre, const bf16 *xbc, SsmView v, uint32_t n, uint32_t start_pos, float *y) {
+__global__ void __launch_bounds__((SC_WARPS + 1) * 32) ssm_chunk_kernel(const float *pre, const bf16 *xbc, SsmView v, uint32_t n, uint32_t start_pos, float *y) {
     using Smem = ChunkSmem<NT>;
+    constexpr int H = NT / 2;  // 16-row tiles of a warp's half of the state
     extern __shared__ __align__(16) uint8_t raw[];
     Smem &sm = *reinterpret_cast<Smem *>(raw);
     const SsmShape &s = v.s;
     pdl_trigger();
     const uint32_t h = blockIdx.x, g = h / (s.heads / s.groups), p0 = blockIdx.y * SC_P, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, N = s.state_p;
     const uint32_t width = min((uint32_t)SC_P, s.dim_p - p0), channels = s.channels(), r = lane >> 2, c2 = (lane & 3) * 2;
+    const uint32_t pw = (warp & 3) * 16, nh = warp >> 2 & 1, n0 = nh * H * 16;  // this warp's values and rows
     const float rate = -expf(v.a_log[h]), dt_bias = v.dt_bias[h], dd = v.d[h];
     pdl_wait();
-    const bool owner = warp * 16 < width;
-    // the state: value p0 + 16 warp + r (+ 8), rows 8 i + c2 (+ 1)
-    float S[2 * NT][4];
-    float *st = v.state + (size_t)h * N * s.dim_p + p0 + warp * 16 + r;
+    auto decays = [&](uint32_t t0, int stage) {  // of the chunk at t0, by one warp: tokens 2 lane, 2 lane + 1
+        float dt[2];
+        double l[2];
 #pragma unroll
-    for (int i = 0; i < 2 * NT; ++i)
+        for (int i = 0; i < 2; ++i) {
+            const uint32_t t = t0 + 2 * lane + i;
+            dt[i] = t < n ? softplus_f32(pre[(size_t)t * s.in_p + s.off_dt() + h] + dt_bias) : 0.0f;  // no token: nothing decays, nothing enters
+            l[i] = (double)(rate * dt[i]);
+        }
+        l[1] += l[0];
+        double before = l[1];
+#pragma unroll
+        for (int o = 1; o < 32; o *= 2) {
+            const double u = __shfl_up_sync(0xffffffffu, before, o);
+            if (lane >= (uint32_t)o) before += u;
+        }
+        const double end = __shfl_sync(0xffffffffu, before, 31);
+        before -= l[1];
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+            const double d = before + l[i];
+            const uint32_t t = 2 * lane + i;
+            sm.l_hi[stage][t] = (float)d;
+            sm.l_lo[stage][t] = (float)(d - (double)(float)d);
+            sm.dt[stage][t] = dt[i];
+            sm.w[stage][t] = expf((float)(end - d)) * dt[i];
+            sm.e[stage][t] = expf((float)d);
+        }
+        if (lane == 0) sm.e_end[stage] = expf((float)end);
+    };
+    if (warp == SC_WARPS) {
+        decays(0, 0);
+        int stage = 0;
+        for (uint32_t t0 = 0; t0 < n; t0 += SC_Q, stage ^= 1) {
+            __syncthreads();
+            if (t0 + SC_Q < n) decays(t0 + SC_Q, stage ^ 1);
+            __syncthreads();
+        }
+        return;
+    }
+    const bool owner = pw < width;
+    // the state: value p0 + pw + r (+ 8), rows n0 + 8 i + c2 (+ 1)
+    float S[2 * H][4];
+    float *st = v.state + ((size_t)h * N + n0) * s.dim_p + p0 + pw + r;
+#pragma unroll
+    for (int i = 0; i < 2 * H; ++i)
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
             const uint32_t row = i * 8 + c2 + (e & 1);
-            S[i][e] = owner && row < N ? st[(size_t)row * s.dim_p + (e >> 1) * 8] : 0.0f;
+            S[i][e] = owner && n0 + row < N ? st[(size_t)row * s.dim_p + (e >> 1) * 8] : 0.0f;
         }
     auto fetch = [&](uint32_t t0, int stage) {
         auto rows = [&](bf16 *dst, uint32_t ld, uint32_t vecs, uint32_t live, uint32_t from) {
@@ -60,80 +105,32 @@ __global__ void __launch_bounds__(SC_WARPS * 32) ssm_chunk_kernel(const float *p
         rows(&sm.x[stage][0][0], SC_LD, SC_P / 8, width, h * s.dim_p + p0);
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
-    float raw_dt[2] = {0.0f, 0.0f};  // of the last warp: tokens 2 lane, 2 lane + 1 of the next chunk
-    auto fetch_dt = [&](uint32_t t0) {
-#pragma unroll
-        for (int i = 0; i < 2; ++i) {
-            const uint32_t t = t0 + 2 * lane + i;
-            if (t < n) raw_dt[i] = pre[(size_t)t * s.in_p + s.off_dt() + h];
-        }
-    };
     fetch(0, 0);
-    if (warp == SC_WARPS - 1) fetch_dt(0);
+    const uint32_t k_row = (lane & 7) + ((lane >> 3) & 1) * 8, k_col = (lane >> 4) * 8;  // of a transposed 16 x 16 operand tile
+    // token tiles: the first two this warp finishes, the others its partner; five tiles of M either way
+    const uint32_t mts[4] = {nh ? 1u : 0u, nh ? 2u : 3u, nh ? 0u : 1u, nh ? 3u : 2u};
     int stage = 0;
     for (uint32_t t0 = 0; t0 < n; t0 += SC_Q, stage ^= 1) {
         asm volatile("cp.async.wait_group 0;" ::: "memory");
         __syncthreads();
         if (t0 + SC_Q < n) fetch(t0 + SC_Q, stage ^ 1);
         const bf16 *bs = &sm.b[stage][0][0], *cs = &sm.c[stage][0][0], *xs = &sm.x[stage][0][0];
-        if (warp == SC_WARPS - 1) {
-            float dt[2];
-            double l[2];
-#pragma unroll
-            for (int i = 0; i < 2; ++i) {
-                dt[i] = t0 + 2 * lane + i < n ? softplus_f32(raw_dt[i] + dt_bias) : 0.0f;  // no token: nothing decays, nothing enters
-                l[i] = (double)(rate * dt[i]);
-            }
-            l[1] += l[0];
-            double before = l[1];
-#pragma unroll
-            for (int o = 1; o < 32; o *= 2) {
-                const double u = __shfl_up_sync(0xffffffffu, before, o);
-                if (lane >= (uint32_t)o) before += u;
-            }
-            const double end = __shfl_sync(0xffffffffu, before, 31);
-            before -= l[1];
-#pragma unroll
-            for (int i = 0; i < 2; ++i) {
-                const double d = before + l[i];
-                const uint32_t t = 2 * lane + i;
-                sm.l_hi[t] = (float)d;
-                sm.l_lo[t] = (float)(d - (double)(float)d);
-                sm.dt[t] = dt[i];
-                sm.w[t] = expf((float)(end - d)) * dt[i];
-                sm.e[t] = expf((float)d);
-            }
-            if (lane == 0) sm.e_end = expf((float)end);
-            fetch_dt(t0 + SC_Q);
-        }
-        // C_t . B_j for the ten 16 x 16 tiles on and below the diagonal, three or two a warp
-        float gt[3][2][4];
-#pragma unroll
-        for (int k = 0; k < 3; ++k) {
-            const uint32_t tile = warp + k * SC_WARPS;
-            if (tile >= 10) continue;
+        const float *l_hi = sm.l_hi[stage], *l_lo = sm.l_lo[stage], *dts = sm.dt[stage], *ws = sm.w[stage], *es = sm.e[stage];
+        // M: C_t . B_j with its weight, for the ten 16 x 16 tiles on and below the diagonal
+#pragma unroll 1
+        for (uint32_t tile = warp; tile < 10; tile += SC_WARPS) {
             const uint32_t mt = tile < 1 ? 0 : tile < 3 ? 1 : tile < 6 ? 2 : 3, nt = tile - mt * (mt + 1) / 2;
             const bf16 *ca = cs + (size_t)(mt * 16 + (lane & 15)) * Smem::LD + (lane >> 4) * 8;
             const bf16 *bb = bs + (size_t)(nt * 16 + (lane & 7) + (lane >> 4) * 8) * Smem::LD + ((lane >> 3) & 1) * 8;
-#pragma unroll
-            for (int q = 0; q < 2; ++q)
-#pragma unroll
-                for (int e = 0; e < 4; ++e) gt[k][q][e] = 0.0f;
+            float gt[2][4] = {};
 #pragma unroll
             for (int kk = 0; kk < NT; ++kk) {
                 uint32_t a[4], b[4];
                 ldsm4(a, ca + kk * 16);
                 ldsm4(b, bb + kk * 16);
-                mma_bf16(gt[k][0], a, b[0], b[1]);
-                mma_bf16(gt[k][1], a, b[2], b[3]);
+                mma_bf16(gt[0], a, b[0], b[1]);
+                mma_bf16(gt[1], a, b[2], b[3]);
             }
-        }
-        __syncthreads();
-#pragma unroll
-        for (int k = 0; k < 3; ++k) {
-            const uint32_t tile = warp + k * SC_WARPS;
-            if (tile >= 10) continue;
-            const uint32_t mt = tile < 1 ? 0 : tile < 3 ? 1 : tile < 6 ? 2 : 3, nt = tile - mt * (mt + 1) / 2;
 #pragma unroll
             for (int q = 0; q < 2; ++q)
 #pragma unroll
@@ -142,123 +139,132 @@ __global__ void __launch_bounds__(SC_WARPS * 32) ssm_chunk_kernel(const float *p
                     float m[2];
 #pragma unroll
                     for (int e = 0; e < 2; ++e)
-                        m[e] = j + e <= t ? gt[k][q][2 * i + e] * expf((sm.l_hi[t] - sm.l_hi[j + e]) + (sm.l_lo[t] - sm.l_lo[j + e])) * sm.dt[j + e] : 0.0f;
+                        m[e] = j + e <= t ? gt[q][2 * i + e] * expf((l_hi[t] - l_hi[j + e]) + (l_lo[t] - l_lo[j + e])) * dts[j + e] : 0.0f;
                     uint32_t hi, lo;
                     split_bf16(m[0], m[1], hi, lo);
                     *reinterpret_cast<uint32_t *>(&sm.m[0][t][j]) = hi;
                     *reinterpret_cast<uint32_t *>(&sm.m[1][t][j]) = lo;
                 }
         }
-#pragma unroll 4
-        for (uint32_t i = threadIdx.x; i < SC_Q * SC_P / 2; i += SC_WARPS * 32) {
-            const uint32_t t = i / (SC_P / 2), p = i % (SC_P / 2) * 2;
+#pragma unroll
+        for (int k = 0; k < SC_Q * SC_P / 2 / (SC_WARPS * 32); ++k) {
+            const uint32_t i = threadIdx.x + k * SC_WARPS * 32, t = i / (SC_P / 2), p = i % (SC_P / 2) * 2;
             const float2 x = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162 *>(xs + (size_t)t * SC_LD + p));
             uint32_t hi, lo;
-            split_bf16(sm.w[t] * x.x, sm.w[t] * x.y, hi, lo);
+            split_bf16(ws[t] * x.x, ws[t] * x.y, hi, lo);
             *reinterpret_cast<uint32_t *>(&sm.wx[0][t][p]) = hi;
             *reinterpret_cast<uint32_t *>(&sm.wx[1][t][p]) = lo;
         }
+        // this half of S^T C
+        float acc[4][2][4] = {};
+        if (owner) {
+            const bf16 *ca = cs + (size_t)(lane & 15) * Smem::LD + n0 + (lane >> 4) * 8;
+#pragma unroll
+            for (int kk = 0; kk < H; ++kk) {
+                uint32_t sh[2][2], sl[2][2];  // [values][first or second eight rows]
+#pragma unroll
+                for (int q = 0; q < 2; ++q)
+#pragma unroll
+                    for (int u = 0; u < 2; ++u) split_bf16(S[2 * kk + u][2 * q], S[2 * kk + u][2 * q + 1], sh[q][u], sl[q][u]);
+                uint32_t a[4][4];
+#pragma unroll
+                for (int o = 0; o < 4; ++o) ldsm4(a[o], ca + (size_t)mts[o] * 16 * Smem::LD + kk * 16);
+#pragma unroll
+                for (int o = 0; o < 4; ++o) {
+                    mma_bf16(acc[o][0], a[o], sh[0][0], sh[0][1]);
+                    mma_bf16(acc[o][1], a[o], sh[1][0], sh[1][1]);
+                }
+#pragma unroll
+                for (int o = 0; o < 4; ++o) {
+                    mma_bf16(acc[o][0], a[o], sl[0][0], sl[0][1]);
+                    mma_bf16(acc[o][1], a[o], sl[1][0], sl[1][1]);
+                }
+            }
+#pragma unroll
+            for (int k = 0; k < 4; ++k)
+                sm.half[warp ^ 4][k][lane] = make_float4(acc[2 + (k >> 1)][k & 1][0], acc[2 + (k >> 1)][k & 1][1], acc[2 + (k >> 1)][k & 1][2], acc[2 + (k >> 1)][k & 1][3]);
+        }
         __syncthreads();
         if (!owner) continue;
-        float acc[4][2][4];
+        // the partner's last two tiles are this warp's first two, in the same order
 #pragma unroll
-        for (int mt = 0; mt < 4; ++mt)
+        for (int o = 0; o < 2; ++o) {
+            const float f0 = es[mts[o] * 16 + r], f1 = es[mts[o] * 16 + r + 8];
 #pragma unroll
-            for (int q = 0; q < 2; ++q)
-#pragma unroll
-                for (int e = 0; e < 4; ++e) acc[mt][q][e] = 0.0f;
-        const bf16 *ca = cs + (size_t)(lane & 15) * Smem::LD + (lane >> 4) * 8;
-#pragma unroll
-        for (int kk = 0; kk < NT; ++kk) {
-            uint32_t sh[2][2], sl[2][2];  // [values][first or second eight rows]
-#pragma unroll
-            for (int q = 0; q < 2; ++q)
-#pragma unroll
-                for (int u = 0; u < 2; ++u) split_bf16(S[2 * kk + u][2 * q], S[2 * kk + u][2 * q + 1], sh[q][u], sl[q][u]);
-#pragma unroll
-            for (int mt = 0; mt < 4; ++mt) {
-                uint32_t a[4];
-                ldsm4(a, ca + (size_t)mt * 16 * Smem::LD + kk * 16);
-                mma_bf16(acc[mt][0], a, sh[0][0], sh[0][1]);
-                mma_bf16(acc[mt][1], a, sh[1][0], sh[1][1]);
-                mma_bf16(acc[mt][0], a, sl[0][0], sl[0][1]);
-                mma_bf16(acc[mt][1], a, sl[1][0], sl[1][1]);
-            }
-        }
-        const uint32_t k_row = (lane & 7) + ((lane >> 3) & 1) * 8, k_col = (lane >> 4) * 8;  // of a transposed 16 x 16 operand tile
-#pragma unroll
-        for (int mt = 0; mt < 4; ++mt) {
-#pragma unroll
-            for (int i = 0; i < 2; ++i) {
-                const float f = sm.e[mt * 16 + r + 8 * i];
-#pragma unroll
-                for (int q = 0; q < 2; ++q) {
-                    acc[mt][q][2 * i] *= f;
-                    acc[mt][q][2 * i + 1] *= f;
-                }
+            for (int q = 0; q < 2; ++q) {
+                const float4 u = sm.half[warp][2 * o + q][lane];
+                acc[o][q][0] = (acc[o][q][0] + u.x) * f0;
+                acc[o][q][1] = (acc[o][q][1] + u.y) * f0;
+                acc[o][q][2] = (acc[o][q][2] + u.z) * f1;
+                acc[o][q][3] = (acc[o][q][3] + u.w) * f1;
             }
         }
 #pragma unroll
-        for (int kt = 0; kt < 4; ++kt) {
+        for (uint32_t kt = 0; kt < 4; ++kt) {
             uint32_t b[4];
-            ldsm4_trans(b, xs + (size_t)(kt * 16 + k_row) * SC_LD + warp * 16 + k_col);
+            ldsm4_trans(b, xs + (size_t)(kt * 16 + k_row) * SC_LD + pw + k_col);
 #pragma unroll
-            for (int mt = kt; mt < 4; ++mt) {
-                uint32_t a[4];
+            for (int o = 0; o < 2; ++o) {
+                if (kt > mts[o]) continue;
+                uint32_t a[2][4];
+#pragma unroll
+                for (int part = 0; part < 2; ++part) ldsm4(a[part], &sm.m[part][mts[o] * 16 + (lane & 15)][kt * 16 + (lane >> 4) * 8]);
 #pragma unroll
                 for (int part = 0; part < 2; ++part) {
-                    ldsm4(a, &sm.m[part][mt * 16 + (lane & 15)][kt * 16 + (lane >> 4) * 8]);
-                    mma_bf16(acc[mt][0], a, b[0], b[1]);
-                    mma_bf16(acc[mt][1], a, b[2], b[3]);
+                    mma_bf16(acc[o][0], a[part], b[0], b[1]);
+                    mma_bf16(acc[o][1], a[part], b[2], b[3]);
                 }
             }
         }
 #pragma unroll
-        for (int mt = 0; mt < 4; ++mt)
+        for (int o = 0; o < 2; ++o)
 #pragma unroll
             for (int i = 0; i < 2; ++i) {
-                const uint32_t t = mt * 16 + r + 8 * i;
+                const uint32_t t = mts[o] * 16 + r + 8 * i;
                 if (t0 + t >= n) continue;
 #pragma unroll
                 for (int q = 0; q < 2; ++q) {
-                    const uint32_t p = warp * 16 + q * 8 + c2;
+                    const uint32_t p = pw + q * 8 + c2;
                     const float2 x = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162 *>(xs + (size_t)t * SC_LD + p));
                     *reinterpret_cast<float2 *>(y + (size_t)(t0 + t) * s.inner_p() + h * s.dim_p + p0 + p) =
-                        make_float2(fmaf(dd, x.x, acc[mt][q][2 * i]), fmaf(dd, x.y, acc[mt][q][2 * i + 1]));
+                        make_float2(fmaf(dd, x.x, acc[o][q][2 * i]), fmaf(dd, x.y, acc[o][q][2 * i + 1]));
                 }
             }
-        const float end = sm.e_end;
+        const float end = sm.e_end[stage];
 #pragma unroll
-        for (int i = 0; i < 2 * NT; ++i)
+        for (int i = 0; i < 2 * H; ++i)
 #pragma unroll
             for (int e = 0; e < 4; ++e) S[i][e] *= end;
 #pragma unroll
         for (int kt = 0; kt < 4; ++kt) {
-            uint32_t ah[4], al[4];
-            const uint32_t row = kt * 16 + (lane & 7) + (lane >> 4) * 8, col = warp * 16 + ((lane >> 3) & 1) * 8;
+            uint32_t ah[4], al[4], b[H][4];
+            const uint32_t row = kt * 16 + (lane & 7) + (lane >> 4) * 8, col = pw + ((lane >> 3) & 1) * 8;
             ldsm4_trans(ah, &sm.wx[0][row][col]);
             ldsm4_trans(al, &sm.wx[1][row][col]);
 #pragma unroll
-            for (int i = 0; i < NT; ++i) {
-                uint32_t b[4];
-                ldsm4_trans(b, bs + (size_t)(kt * 16 + k_row) * Smem::LD + i * 16 + k_col);
-                mma_bf16(S[2 * i], ah, b[0], b[1]);
-                mma_bf16(S[2 * i + 1], ah, b[2], b[3]);
-                mma_bf16(S[2 * i], al, b[0], b[1]);
-                mma_bf16(S[2 * i + 1], al, b[2], b[3]);
+            for (int i = 0; i < H; ++i) ldsm4_trans(b[i], bs + (size_t)(kt * 16 + k_row) * Smem::LD + n0 + i * 16 + k_col);
+#pragma unroll
+            for (int i = 0; i < H; ++i) {
+                mma_bf16(S[2 * i], ah, b[i][0], b[i][1]);
+                mma_bf16(S[2 * i + 1], ah, b[i][2], b[i][3]);
+            }
+#pragma unroll
+            for (int i = 0; i < H; ++i) {
+                mma_bf16(S[2 * i], al, b[i][0], b[i][1]);
+                mma_bf16(S[2 * i + 1], al, b[i][2], b[i][3]);
             }
         }
     }
     if (owner) {
 #pragma unroll
-        for (int i = 0; i < 2 * NT; ++i)
+        for (int i = 0; i < 2 * H; ++i)
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
                 const uint32_t row = i * 8 + c2 + (e & 1);
-                if (row < N) st[(size_t)row * s.dim_p + (e >> 1) * 8] = S[i][e];
+                if (n0 + row < N) st[(size_t)row * s.dim_p + (e >> 1) * 8] = S[i][e];
             }
     }
-    ssm_keep(pre, v, h, p0, p0 + width, blockIdx.y == 0, n, start_pos);
+    ssm_keep(pre, v, h, p0, p0 + width, blockIdx.y == 0, n, start_pos, SC_WARPS * 32);
 }
 
 template <int NT>
@@ -267,7 +273,7 @@ int32_t launch_nt(const float *pre, const bf16 *xbc, const SsmView &v, size_t n,
     auto k = ssm_chunk_kernel<NT>;
     CERA_CUDA_TRY(cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, sizeof(ChunkSmem<NT>)));
     count_launch();
-    return check_cuda(launch_k(k, grid, dim3(SC_WARPS * 32), sizeof(ChunkSmem<NT>), st, pre, xbc, v, (uint32_t)n, (uint32_t)start_pos, y), "ssm chunk launch");
+    return check_cuda(launch_k(k, grid, dim3((SC_WARPS + 1) * 32), sizeof(ChunkSmem<NT>), st, pre, xbc, v, (uint32_t)n, (uint32_t)start_pos, y), "ssm chunk launch");
 }
 
 }  // namespace
