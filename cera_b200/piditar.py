@@ -23,7 +23,7 @@ def _layer(i, entry):
         rot = m["rot"]
         d.mixer = Mixer.ATTENTION
         d.n_heads, d.n_kv_heads, d.head_dim, d.value_dim = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
-        d.rot_dim, d.rope_base, d.attn_scale, d.softcap = rot["dims"], rot["base"], m["scale"], m["softcap"]
+        d.rot_dim, d.rope_base, d.attn_scale, d.softcap = rot["dims"], rot["base"], m["scale"], m.get("softcap") or 0.0
         d.qk_norm = d.attn_bias = 1
     elif entry["type"] == "rglru":
         d.mixer = Mixer.RGLRU
@@ -47,9 +47,11 @@ def _layer(i, entry):
 
 def describe(config):
     """config.json (parsed) -> (model keywords, layer descriptions)."""
-    loop = config.get("loop") or {"start": 0, "stop": 0, "times": 1}
+    loop = config.get("loop") or {}
+    start, stop = loop.get("start", 0), loop.get("stop", 0)
     return (dict(hidden_size=config["width"], vocab_size=config["vocab"], norm_eps=config["norm"]["eps"], embedding_scale=config["embedding"]["scale"],
-                 norm_offset=NORM_OFFSET, tied_output=1, no_post_norms=1, loop_start=loop["start"], loop_stop=loop["stop"], loop_times=loop["times"]),
+                 norm_offset=NORM_OFFSET, tied_output=1, no_post_norms=1, loop_start=start, loop_stop=stop,
+                 loop_times=loop["times"] if stop > start else 1),
             [_layer(i, e) for i, e in enumerate(config["layers"])])
 
 

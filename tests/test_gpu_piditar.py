@@ -32,6 +32,7 @@ MECHANISMS = {
     "mamba2_norm_across_heads": [mamba2(heads=6, vdim=20, state=48, groups=3, norm_groups=4, conv=5)],
     "mamba2_wide": [mamba2(heads=4, vdim=64, state=128, groups=1, norm_groups=1)],
     "mamba2_wide_values": [mamba2(heads=2, vdim=130, state=100, groups=2, norm_groups=2, conv=3)],
+    "mamba2_state_200": [mamba2(heads=2, vdim=72, state=200, groups=1)],
     "mamba2_large_state": [mamba2(heads=2, vdim=48, state=300, groups=1)],
     "unit": [rglru(width=8, blocks=1, mlp=unit(200))],
     "unit_narrow": [rglru(width=8, blocks=1, mlp=unit(9))],
