@@ -1,7 +1,7 @@
 // State-space recurrence with a matrix state per head (Mamba-2): S = exp(-exp(A_log) dt) S + dt B x^T, y = S^T C + D x,
 // dt = softplus(raw + bias); x, B, C come convolved through silu, B and C are shared by the heads of a group.  This file: the
-// decode step, the token-by-token scan (f32, short portions, states too large for ssm_chunk.cu) and the gated norm behind all.  States, step sizes and decays are f32; a decay
-// next to 1 enters as its difference from 1.
+// decode step, the token-by-token scan (f32, short portions, states too large for ssm_chunk.cu) and the gated norm behind
+// all.  States, step sizes and decays are f32; a decay next to 1 enters as its difference from 1.
 #include "dense_gemv.cuh"
 #include "ssm.cuh"
 
